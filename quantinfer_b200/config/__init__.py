@@ -5,11 +5,12 @@ from .bebuvik import BebuvikConfig
 from .kiruvik import KiruvikConfig
 from .dulotar import DulotarConfig
 from .lemotar import LemotarConfig
+from .siditar import SiditarConfig
 from .spec import (AttentionSpec, BigramEmbeddingSpec, DenseFeedForwardSpec, EmbeddingSpec, FeedForwardSpec, HeadSpec,
                    LatentAttentionSpec, LayerCall, LayerSpec, ModelSpec, NormSpec, ParallelLayerSpec, PositionSpec,
                    RotarySpec, ShortConvSpec, ClampedGLUSpec, GatedAttentionSpec, MoESpec, ReentrySpec, SandwichLayerSpec,
                    StateSpaceSpec, ConvPreNormLayerSpec, LightningAttentionSpec, MinGRUSpec, ParallelMixersSpec, TimeMixSpec,
-                   GatedDeltaSpec, PostNormLayerSpec)
+                   GatedDeltaSpec, PostNormLayerSpec, GatedLinearAttentionSpec, HyperLayerSpec, StreamSumNormSpec)
 
 __all__ = [
     "Qwen3Config", "architectures", "config_class_for", "config_from_dict", "load_config",
@@ -19,4 +20,5 @@ __all__ = [
     "KiruvikConfig", "ClampedGLUSpec", "GatedAttentionSpec", "MoESpec", "ReentrySpec", "SandwichLayerSpec", "StateSpaceSpec",
     "DulotarConfig", "ConvPreNormLayerSpec", "LightningAttentionSpec", "MinGRUSpec", "ParallelMixersSpec", "TimeMixSpec",
     "LemotarConfig", "GatedDeltaSpec", "PostNormLayerSpec",
+    "SiditarConfig", "GatedLinearAttentionSpec", "HyperLayerSpec", "StreamSumNormSpec",
 ]

@@ -82,6 +82,9 @@ def _register_builtin() -> None:
     from .lemotar import ARCHITECTURE as LEMOTAR, LemotarConfig
 
     register_architecture(LEMOTAR, LemotarConfig)
+    from .siditar import ARCHITECTURE as SIDITAR, SiditarConfig
+
+    register_architecture(SIDITAR, SiditarConfig)
 
 
 _register_builtin()

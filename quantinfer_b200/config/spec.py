@@ -25,7 +25,7 @@ class NormSpec:
     coordinates, the tensor named `prefix` itself, of shape []. "dyt": dynamic tanh, tanh(alpha x) w + b with no
     statistic of the row (eps unused): w is the tensor named `prefix` itself, b `prefix + ".b"`, alpha
     `prefix + ".alpha"` of shape []. "layernorm": (x - mean) / sqrt(variance + eps) * w + b with the variance the mean
-    squared deviation; w is the tensor named `prefix` itself, b `prefix + ".b"`."""
+    squared deviation; w is the tensor named `prefix` itself, b `prefix + ".b"`. "layernorm_nobias": the same without b."""
 
     size: int
     eps: float
@@ -207,7 +207,12 @@ class GatedAttentionSpec:
                                        # value: "zero": b_h = 0 (one is added); "learned": b is the tensor `sink` [heads]
     values_from_keys: bool = False     # there is no `v`: a position's value is its key as projected (before any norm and
                                        # rotation), so value_dim equals head_dim
-    qk_norm: Optional[str] = None      # "whole": q (all heads at once) and k (likewise) each pass one RMS norm over the whole
+    q_temp: Optional[tuple] = None     # (coef, every): q is multiplied by 1 + coef ln(floor((p + 1) / every) + 1) at position p
+    distance_bias: Optional[float] = None  # D: a key n positions back adds a learned number per head to its score (after scale and
+                                       # cap), row bucket(n) of the table `rel` [rows, heads]: a row a distance below rows / 2, the
+                                       # other rows over distances that grow geometrically up to D
+    qk_norm: Optional[str] = None      # "head": every head of q and k passes an RMS norm of its own before the rotation, gains
+                                       # `q.norm`, `k.norm` [head_dim] that the heads share. "whole": q (all heads at once) and k (likewise) each pass one RMS norm over the whole
                                        # projection before the rotation, gains `q.norm` [heads head_dim], `k.norm`
     qk_norm_eps: float = 1e-6
 
@@ -275,6 +280,7 @@ class ParallelMixersSpec:
     out_norm_eps: float = 1e-6
     sum_scale: float = 1.0
     hidden_size: Optional[int] = None  # needed with `out_norm_names` (the gains' size)
+    branch_scales: Optional[tuple] = None  # (left, right): factors on the two outputs, without norms: left * a + right * b
 
 
 @dataclass(frozen=True)
@@ -298,6 +304,49 @@ class GatedDeltaSpec:
     unit_eps: float = 1e-6
     prefix: str = ""
     kind: str = "gated_delta"
+
+
+@dataclass(frozen=True)
+class GatedLinearAttentionSpec:
+    """Linear attention over a matrix state per head whose decay per key channel is a gate of the token: q = W_q x
+    head_dim^(-1/2), k = W_k x (`heads` x `head_dim`), v = W_v x (`heads` x `value_dim`); decay = sigmoid(W_a2 W_a1 x +
+    b)^(1 / `tau`) (`a1` [rank, hidden], `a2` [heads head_dim, rank], `a2.b`; the rank is read from `a1`); S_t =
+    diag(decay_t) S_(t-1) + k_t v_t^T; o_t = S_t^T q_t; every head's o over its root mean square times `norm`
+    [value_dim], times silu(W_g x), W_o. State (32-bit): S."""
+
+    hidden_size: int
+    heads: int
+    head_dim: int
+    value_dim: int
+    tau: float
+    norm_eps: float
+    prefix: str = ""
+    kind: str = "gated_linear_attention"
+
+
+@dataclass(frozen=True)
+class HyperLayerSpec:
+    """The block of a model with residual streams x_1 .. x_s (hyper-connections). For each sublayer (mixer, then feed-forward,
+    which may be absent) with its tensors `<name>.in` [s], `<name>.out` [s], `<name>.mix` [s, s]: u = sum_s in_s x_s; y =
+    sublayer(norm(u)); then, all streams at once, x_t <- sum_s mix[s, t] x_s + out_t y. `names`: the prefixes of the two
+    sublayers' tensors."""
+
+    mixer_norm: NormSpec
+    mixer: object
+    ffn_norm: Optional[NormSpec]
+    ffn: object
+    streams: int
+    names: tuple
+    kind: str = "hyper"
+
+
+@dataclass(frozen=True)
+class StreamSumNormSpec:
+    """A norm of the sum of the residual streams (the final norm of a model that has several)."""
+
+    norm: NormSpec
+    streams: int
+    kind: str = "stream_sum"
 
 
 @dataclass(frozen=True)
@@ -434,6 +483,8 @@ class EmbeddingSpec:
     kind: str = "embedding"
     weight_name: Optional[str] = None   # the tensor's full name when it is not prefix + "weight"
     scale: float = 1.0                  # the row is multiplied by this (32-bit) on its way into the stream
+    sinusoid_base: Optional[float] = None   # b: the position vector sin(p b^(-2i / hidden)), cos(...) (interleaved) is added
+    copies: int = 1                     # residual streams that all start as this row, side by side
 
 
 @dataclass(frozen=True)

@@ -9,7 +9,8 @@
 // with lo = 0, or p - window + 1 for a windowed layer, or the start of p's chunk
 // (floor(p / chunk) * chunk, chunks counted from the sequence's first position)
 // for a chunked layer; both bounds may hold at once. A soft cap c replaces each
-// score by c tanh(score / c) before the softmax. Values may have another
+// score by c tanh(score / c) before the softmax; a distance bias then adds a number per
+// head that depends on p - j alone. Values may have another
 // size `dv` than queries and keys, and the result may be multiplied, element by
 // element, by the sigmoid of a gate row (an output gate computed from the
 // mixer's input). Scores, the maximum,
@@ -37,7 +38,8 @@ attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const T* 
                          int max_blocks, int page_size, int num_pages,
                          const int* __restrict__ positions, const int* __restrict__ token_req,
                          int nq, int nkv, int d, int dv, float scale, float softcap, float out_scale, int window, int chunk,
-                         const T* __restrict__ gate, long long ldg, const float* __restrict__ sink, int* __restrict__ status) {
+                         const T* __restrict__ gate, long long ldg, const float* __restrict__ sink, const float* __restrict__ bias, int bias_len,
+                         int* __restrict__ status) {
     extern __shared__ float smem[];
     float* q_s = smem;                          // [d]
     float* part_acc = smem + d;                 // [kWarps][dv]
@@ -78,6 +80,7 @@ attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const T* 
                 for (int i = 0; i < d; ++i) dot = fmaf(q_s[i], qi::to_f32<T>(krow[i]), dot);
                 s = dot * scale;
                 if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+                if (bias) s += bias[(size_t)h * bias_len + min(pos - j, bias_len - 1)];
             }
         }
         const float cm = qi::warp_max(s);
@@ -143,12 +146,15 @@ attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const T* 
 // window 0: no window; chunk 0: no chunks; gate (may be null): row t, head h, element i at gate[t * ldg + h * dv + i];
 // softcap c > 0: a score s becomes c tanh(s / c) before the softmax (0: scores as they are); out_scale multiplies the result.
 // sink (may be null): float32 [nq]; the softmax's denominator of head h holds exp(sink[h]) once more.
-extern "C" int qi_attention_generic_sink(const void* q, void* out, int dtype, const void* k_pages,
+// bias (may be null): float32 [nq, bias_len]; a key n positions back adds bias[h, min(n, bias_len - 1)] to its score.
+extern "C" int qi_attention_generic_bias(const void* q, void* out, int dtype, const void* k_pages,
                                        const void* v_pages, const int* block_table, int max_blocks,
                                        int page_size, int num_pages, const int* positions,
                                        const int* token_req, int n_tokens, int nq, int nkv, int d, int dv,
                                        float scale, float softcap, float out_scale, int window, int chunk, const void* gate,
-                                       long long ldg, const float* sink, int* status, cudaStream_t stream) {
+                                       long long ldg, const float* sink, const float* bias, int bias_len, int* status,
+                                       cudaStream_t stream) {
+    QI_REQUIRE(!bias || bias_len > 0, "attention: an empty distance bias");
     QI_REQUIRE(n_tokens >= 0 && nq > 0 && nkv > 0 && d > 0 && dv > 0, "attention: bad sizes");
     QI_REQUIRE(nq % nkv == 0, "attention: %d query heads are not a multiple of %d kv heads", nq, nkv);
     QI_REQUIRE(d <= kMaxD && dv <= kMaxD, "attention: head sizes %d / %d are above the limit %d of this kernel", d, dv, kMaxD);
@@ -168,10 +174,21 @@ extern "C" int qi_attention_generic_sink(const void* q, void* out, int dtype, co
                 (const T*)q + (size_t)t0 * nq * d, (T*)out + (size_t)t0 * nq * dv, (const T*)k_pages,
                 (const T*)v_pages, block_table, max_blocks, page_size, num_pages, positions + t0,
                 token_req + t0, nq, nkv, d, dv, scale, softcap, out_scale, window, chunk,
-                gate ? (const T*)gate + (size_t)t0 * ldg : (const T*)nullptr, ldg, sink, status);
+                gate ? (const T*)gate + (size_t)t0 * ldg : (const T*)nullptr, ldg, sink, bias, bias_len, status);
         });
     }
     return qi::check_launch("attention_generic");
+}
+
+extern "C" int qi_attention_generic_sink(const void* q, void* out, int dtype, const void* k_pages,
+                                       const void* v_pages, const int* block_table, int max_blocks,
+                                       int page_size, int num_pages, const int* positions,
+                                       const int* token_req, int n_tokens, int nq, int nkv, int d, int dv,
+                                       float scale, float softcap, float out_scale, int window, int chunk, const void* gate,
+                                       long long ldg, const float* sink, int* status, cudaStream_t stream) {
+    return qi_attention_generic_bias(q, out, dtype, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, positions,
+                                     token_req, n_tokens, nq, nkv, d, dv, scale, softcap, out_scale, window, chunk, gate, ldg,
+                                     sink, nullptr, 0, status, stream);
 }
 
 extern "C" int qi_attention_generic_cap(const void* q, void* out, int dtype, const void* k_pages,

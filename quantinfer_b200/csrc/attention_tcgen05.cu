@@ -264,7 +264,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                                       float scale_log2e, int window, int* __restrict__ status, int n_ranges,
                                       float* __restrict__ ws_o, float* __restrict__ ws_ml, int chunk,
                                       const qi::bf16* __restrict__ gate, long long ldg, float cap, float cap_pre,
-                                      float out_scale, const float* __restrict__ sink) {
+                                      float out_scale, const float* __restrict__ sink, const float* __restrict__ bias, int bias_len) {
     extern __shared__ uint8_t smem_raw[];
     using B = Bars;
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -490,10 +490,27 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                     sv[c] = __float_as_uint(fmaf(-cap, __fdividef(2.f, 1.f + t), cap));
                 }
             }
+            // the distance bias (base 2, natural numbers in the table): a warp whose rows are all beyond its reach shifts the
+            // tile's exponents by one number, at no cost a score; a nearer one reads an entry a score (neighbouring lanes
+            // read neighbouring entries of a table of a few KB, from the first-level cache)
+            float sc = scale_log2e, shift = 0.f;
+            if (bias) {
+                const float* bh = bias + (size_t)h * bias_len;
+                if (pos0 + quarter * 32 - (t0 + BN - 1) >= bias_len - 1) {
+                    shift = __ldg(bh + bias_len - 1) * 1.4426950408889634f;
+                } else {
+                    sc = 1.f;
+#pragma unroll
+                    for (int c = 0; c < BN; ++c) {
+                        const float b = __ldg(bh + min(max(pos - t0 - c, 0), bias_len - 1));
+                        sv[c] = __float_as_uint(fmaf(b, 1.4426950408889634f, __uint_as_float(sv[c]) * scale_log2e));
+                    }
+                }
+            }
             // a tile that lies wholly inside every row's span takes the code without the comparisons
             const bool interior = __all_sync(0xffffffffu, c_lo == 0 && c_hi == BN);
             const float mx = interior ? row_max<false>(sv, 0, BN) : row_max<true>(sv, c_lo, c_hi);
-            const float m_top = fmaxf(m, mx * scale_log2e);
+            const float m_top = fmaxf(m, fmaf(mx, sc, shift));
             const bool fresh = m == -INFINITY;
             const bool moves = !fresh && m_top - m > kRescaleStep;
             if (__any_sync(0xffffffffu, moves)) {
@@ -518,8 +535,8 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
             const float ms = (m == -INFINITY) ? 0.f : m;
             if (u > 1 && !mbar_wait(bars + B::p_free + 8 * (u & 1u), ((u >> 1) & 1u) ^ 1u, abort_flag)) { ok = false; break; }   // P.V of tile j - 2 has read this buffer
             uint32_t pk[BN / 2];
-            const float sum = interior ? row_weights<false>(sv, pk, scale_log2e, ms, 0, BN)
-                                       : row_weights<true>(sv, pk, scale_log2e, ms, c_lo, c_hi);
+            const float sum = interior ? row_weights<false>(sv, pk, sc, ms - shift, 0, BN)
+                                       : row_weights<true>(sv, pk, sc, ms - shift, c_lo, c_hi);
             l += sum;
             tmem_st32(tmem_p + (u & 1u) * 32 + lane_addr, pk);
             tmem_st_wait();
@@ -671,14 +688,16 @@ extern "C" int qi_attention_prefill_tcgen05_supported(int nq, int nkv, int d, in
 // key j <= i only if floor(i / chunk) = floor(j / chunk). gate (or null): bfloat16 [n_tokens, nq * 128] with rows
 // `ldg` elements apart; the output is multiplied element by element with its sigmoid. softcap c > 0: a score s (scale
 // applied) becomes c tanh(s / c) before the softmax. out_scale multiplies the result. sink (or null): float32 [nq]; the
-// softmax's denominator of head h holds exp(sink[h]) once more.
-extern "C" int qi_attention_prefill_tcgen05_sink(const void* q, void* out, const void* k_pages, const void* v_pages,
+// softmax's denominator of head h holds exp(sink[h]) once more. bias (or null): float32 [nq, bias_len]; a key n positions
+// back adds bias[h, min(n, bias_len - 1)] to its score (after the cap).
+extern "C" int qi_attention_prefill_tcgen05_bias(const void* q, void* out, const void* k_pages, const void* v_pages,
                                                const int* block_table, int max_blocks, int page_size, int num_pages,
                                                const int* q_start, const int* start_pos, const int* tile_req,
                                                const int* tile_q0, int n_tiles, int n_tokens, int nq, int nkv, int d,
                                                float scale, int window, int chunk, const void* gate, long long ldg,
                                                int n_ranges, float* workspace, int* status, float softcap, float out_scale,
-                                               const float* sink, cudaStream_t stream) {
+                                               const float* sink, const float* bias, int bias_len, cudaStream_t stream) {
+    QI_REQUIRE(!bias || bias_len > 0, "attention_prefill_tcgen05: an empty distance bias");
     QI_REQUIRE(softcap >= 0.f && scale > 0.f, "attention_prefill_tcgen05: the soft cap must be >= 0 (0 = none) and the scale positive");
     QI_REQUIRE(chunk >= 0 && (!gate || (((uintptr_t)gate & 15) == 0 && ldg % 8 == 0 && ldg >= (long long)nq * D)),
                "attention_prefill_tcgen05: a gate must be 16-byte aligned with rows a multiple of 8 elements apart");
@@ -712,7 +731,7 @@ extern "C" int qi_attention_prefill_tcgen05_sink(const void* q, void* out, const
     qi::launch(attention_prefill_tcgen05_kernel, dim3(nq, n_tiles, n_ranges), dim3(kThreads), kSmemBytes, stream, mq, mk, mv,
                (qi::bf16*)out, block_table, max_blocks, page_size, box_rows, num_pages, q_start, start_pos, tile_req,
                tile_q0, nq, nkv, softcap > 0.f ? log2e : scale * log2e, window, status, n_ranges, ws_o, ws_ml, chunk,
-               (const qi::bf16*)gate, ldg, softcap, cap_pre, out_scale, sink);
+               (const qi::bf16*)gate, ldg, softcap, cap_pre, out_scale, sink, bias, bias_len);
     if (n_ranges > 1) {
         if (int rc = qi::check_launch("attention_prefill_tcgen05")) return rc;
         qi::launch(attention_prefill_merge_kernel, dim3(nq, n_tokens), dim3(128), 0, stream, (const float*)ws_o,
@@ -729,9 +748,9 @@ extern "C" int qi_attention_prefill_tcgen05_ex(const void* q, void* out, const v
                                                float scale, int window, int chunk, const void* gate, long long ldg,
                                                int n_ranges, float* workspace, int* status, float softcap, float out_scale,
                                                cudaStream_t stream) {
-    return qi_attention_prefill_tcgen05_sink(q, out, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, q_start,
+    return qi_attention_prefill_tcgen05_bias(q, out, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, q_start,
                                              start_pos, tile_req, tile_q0, n_tiles, n_tokens, nq, nkv, d, scale, window, chunk,
-                                             gate, ldg, n_ranges, workspace, status, softcap, out_scale, nullptr, stream);
+                                             gate, ldg, n_ranges, workspace, status, softcap, out_scale, nullptr, nullptr, 0, stream);
 }
 
 extern "C" int qi_attention_prefill_tcgen05(const void* q, void* out, const void* k_pages, const void* v_pages,

@@ -111,3 +111,52 @@ extern "C" int qi_embedding_bigram(const void* table, const void* bigram, int ta
     });
     return qi::check_launch("embedding_bigram");
 }
+
+// Embedding with a sinusoidal position vector: for every copy c of a token's row
+//     out[t, c, i] = table[ids[t], i] * scale + (i even ? sin : cos)(positions[t] * freq[i / 2])
+// The angle is formed and reduced to one turn in 64-bit (a position of a few thousand in 32-bit would leave an error of
+// 1e-4 in it), sine and cosine are 32-bit. `copies` writes the row that many times side by side (residual streams).
+namespace {
+
+template <typename TW>
+__global__ void embedding_sinusoid_kernel(const TW* __restrict__ table, const int* __restrict__ ids, const int* __restrict__ positions,
+                                          const double* __restrict__ freq, float* __restrict__ out, int hidden, int vocab, int copies,
+                                          float scale, int* __restrict__ status) {
+    qi::pdl_wait();
+    const int t = blockIdx.x;
+    const int id = ids[t];
+    const bool known = id >= 0 && id < vocab;
+    if (!known && threadIdx.x == 0 && status) atomicOr(status, qi::kStatusBadToken);
+    float* dst = out + (size_t)t * copies * hidden;
+    const TW* src = table + (size_t)(known ? id : 0) * hidden;
+    const double pos = (double)positions[t], turn = 6.283185307179586476925;
+    for (int pair = threadIdx.x; 2 * pair < hidden; pair += blockDim.x) {
+        const double angle = pos * freq[pair];
+        float sn, cs;
+        sincosf((float)(angle - turn * rint(angle / turn)), &sn, &cs);
+        const int i = 2 * pair;
+        const float a = known ? fmaf(qi::to_f32<TW>(src[i]), scale, sn) : 0.f;
+        const float b = known && i + 1 < hidden ? fmaf(qi::to_f32<TW>(src[i + 1]), scale, cs) : 0.f;
+        for (int c = 0; c < copies; ++c) {
+            dst[(size_t)c * hidden + i] = a;
+            if (i + 1 < hidden) dst[(size_t)c * hidden + i + 1] = b;
+        }
+    }
+}
+
+}  // namespace
+
+// freq float64 [ceil(hidden / 2)]; out float32 [n_tokens, copies, hidden].
+extern "C" int qi_embedding_sinusoid(const void* table, int table_dtype, const int* ids, const int* positions, const double* freq,
+                                     float* out, int n_tokens, int hidden, int vocab, int copies, float scale, int* status,
+                                     cudaStream_t stream) {
+    QI_REQUIRE(n_tokens >= 0 && hidden > 0 && vocab > 0 && copies > 0, "embedding_sinusoid: bad sizes n=%d hidden=%d vocab=%d copies=%d",
+               n_tokens, hidden, vocab, copies);
+    if (n_tokens == 0) return 0;
+    const int threads = hidden >= 1024 ? 256 : (hidden >= 256 ? 128 : 64);
+    QI_DISPATCH_DTYPE(table_dtype, TW, {
+        qi::launch(embedding_sinusoid_kernel<TW>, dim3(n_tokens), dim3(threads), 0, stream, (const TW*)table, ids, positions, freq, out,
+                   hidden, vocab, copies, scale, status);
+    });
+    return qi::check_launch("embedding_sinusoid");
+}

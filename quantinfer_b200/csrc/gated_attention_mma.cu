@@ -6,6 +6,8 @@
 //     s_ij = cap((q_i . k_j) * scale)    for lo(i) <= j <= i,   lo(i) = max(start of i's chunk, i - window + 1, 0)
 //     out_i = (sum_j softmax(s_i)_j v_j) * sigmoid(gate_i) * out_scale      cap(s) = c tanh(s / c), or s without a cap
 //
+// A distance bias (optional) adds to s_ij a number per head that depends on i - j alone (after the cap).
+//
 // One kernel serves prompts, portions and single decode tokens: a CTA of four warps takes up to 64
 // consecutive query rows of ONE step entry and one query head (the tiles are found on the device from
 // q_start, so the launch can sit in a CUDA graph), walks the keys its rows can see in tiles of 64 that
@@ -73,7 +75,7 @@ gated_attention_mma_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restrict_
                            int page_size, int num_pages, const int* __restrict__ q_start, const int* __restrict__ start_pos,
                            int n_entries, int nq, int nkv, int d, int dv, float scale_log2e, float softcap, float out_scale,
                            int window, int chunk, const qi::bf16* __restrict__ gate, long long ldg, const float* __restrict__ sink,
-                           int n_ranges, float* __restrict__ ws_o, float* __restrict__ ws_ml, int* __restrict__ status) {
+                           const float* __restrict__ bias, int bias_len, int n_ranges, float* __restrict__ ws_o, float* __restrict__ ws_ml, int* __restrict__ status) {
     extern __shared__ __align__(16) uint8_t smem_raw[];
     constexpr int SK = DK + kPad, SV = DV + kPad;
     qi::bf16* Qs = reinterpret_cast<qi::bf16*>(smem_raw);       // [kQT][SK]
@@ -184,6 +186,28 @@ gated_attention_mma_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restrict_
                 for (int j = 0; j < 4; ++j) s[n][j] = b * tanhf(s[n][j] * a);
             }
         }
+        // the distance bias: tiles beyond its reach take one number, nearer ones an entry a score (cached: a head's table is
+        // a few KB, and a warp's scores of one instruction read at most 15 neighbouring entries)
+        float add = 0.f;
+        bool near = false;
+        if (bias) {
+            if (pos0 - (t0 + kKT - 1) >= bias_len - 1) {
+                add = bias[(size_t)h * bias_len + bias_len - 1] * 1.4426950408889634f;
+            } else {
+                near = true;
+                const float* bh = bias + (size_t)h * bias_len;
+#pragma unroll
+                for (int n = 0; n < kKT / 8; ++n) {
+#pragma unroll
+                    for (int j = 0; j < 2; ++j) {
+                        const int key = t0 + n * 8 + (lane & 3) * 2 + j;
+                        s[n][j] = s[n][j] * scale_log2e + __ldg(bh + min(max(pA - key, 0), bias_len - 1)) * 1.4426950408889634f;
+                        s[n][2 + j] = s[n][2 + j] * scale_log2e + __ldg(bh + min(max(pB - key, 0), bias_len - 1)) * 1.4426950408889634f;
+                    }
+                }
+            }
+        }
+        const float mul = near ? 1.f : scale_log2e;
         // mask, scale (into the base-2 exponent), row maxima
         float tmA = -INFINITY, tmB = -INFINITY;
 #pragma unroll
@@ -191,8 +215,8 @@ gated_attention_mma_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restrict_
 #pragma unroll
             for (int j = 0; j < 2; ++j) {
                 const int key = t0 + n * 8 + (lane & 3) * 2 + j;
-                s[n][j] = (key >= loA && key <= pA && rA < rows) ? s[n][j] * scale_log2e : -INFINITY;
-                s[n][2 + j] = (key >= loB && key <= pB && rB < rows) ? s[n][2 + j] * scale_log2e : -INFINITY;
+                s[n][j] = (key >= loA && key <= pA && rA < rows) ? fmaf(s[n][j], mul, add) : -INFINITY;
+                s[n][2 + j] = (key >= loB && key <= pB && rB < rows) ? fmaf(s[n][2 + j], mul, add) : -INFINITY;
                 tmA = fmaxf(tmA, s[n][j]);
                 tmB = fmaxf(tmB, s[n][2 + j]);
             }
@@ -319,7 +343,7 @@ template <int DK, int DV>
 int launch_one(dim3 grid, cudaStream_t stream, const void* q, void* out, const void* k_pages, const void* v_pages,
                const int* block_table, int max_blocks, int page_size, int num_pages, const int* q_start, const int* start_pos,
                int n_entries, int nq, int nkv, int d, int dv, float scale_log2e, float softcap, float out_scale, int window, int chunk,
-               const void* gate, long long ldg, const float* sink, int n_ranges, float* ws_o, float* ws_ml, int n_tokens, int* status) {
+               const void* gate, long long ldg, const float* sink, const float* bias, int bias_len, int n_ranges, float* ws_o, float* ws_ml, int n_tokens, int* status) {
     const size_t smem = sizeof(qi::bf16) * ((size_t)(kQT + 2 * kKT) * (DK + kPad) + (size_t)2 * kKT * (DV + kPad));
     static bool raised = false;
     if (!raised && smem > 48 * 1024) {
@@ -328,7 +352,7 @@ int launch_one(dim3 grid, cudaStream_t stream, const void* q, void* out, const v
     }
     qi::launch(gated_attention_mma_kernel<DK, DV>, grid, dim3(kThreads), smem, stream, (const qi::bf16*)q, (qi::bf16*)out,
                (const qi::bf16*)k_pages, (const qi::bf16*)v_pages, block_table, max_blocks, page_size, num_pages, q_start, start_pos,
-               n_entries, nq, nkv, d, dv, scale_log2e, softcap, out_scale, window, chunk, (const qi::bf16*)gate, ldg, sink, n_ranges, ws_o, ws_ml, status);
+               n_entries, nq, nkv, d, dv, scale_log2e, softcap, out_scale, window, chunk, (const qi::bf16*)gate, ldg, sink, bias, bias_len, n_ranges, ws_o, ws_ml, status);
     if (n_ranges > 1) {
         if (int rc = qi::check_launch("gated_attention_mma")) return rc;
         qi::launch(gated_attention_merge_kernel, dim3(nq, n_tokens), dim3(128), 0, stream, (const float*)ws_o, (const float*)ws_ml,
@@ -348,13 +372,16 @@ extern "C" int qi_gated_attention_mma_supported(int nq, int nkv, int d, int dv) 
 // start_pos [entries]; gate (may be null) row t, head h, element i at gate[t * ldg + h * dv + i] (ldg and dv even);
 // softcap c > 0: a score s becomes c tanh(s / c) before the softmax; out_scale multiplies the result. sink (may be null):
 // float32 [nq]; the softmax's denominator of head h holds exp(sink[h]) once more.
+// bias (may be null): float32 [nq, bias_len]; a key n positions back adds bias[h, min(n, bias_len - 1)] to its score.
 // n_ranges > 1 (steps of single tokens over long contexts): every query tile's keys are cut into that many ranges over
 // separate CTAs and a second kernel adds the parts; `workspace` must then hold n_tokens * nq * n_ranges * (dv + 2) floats.
-extern "C" int qi_gated_attention_mma_ranges(const void* q, void* out, const void* k_pages, const void* v_pages, const int* block_table,
+extern "C" int qi_gated_attention_mma_bias(const void* q, void* out, const void* k_pages, const void* v_pages, const int* block_table,
                                       int max_blocks, int page_size, int num_pages, const int* q_start, const int* start_pos,
                                       int n_entries, int n_tokens, int nq, int nkv, int d, int dv, float scale, float softcap,
                                       float out_scale, int window, int chunk, const void* gate, long long ldg, const float* sink,
-                                      int n_ranges, float* workspace, int* status, cudaStream_t stream) {
+                                      const float* bias, int bias_len, int n_ranges, float* workspace, int* status,
+                                      cudaStream_t stream) {
+    QI_REQUIRE(!bias || bias_len > 0, "gated_attention_mma: an empty distance bias");
     QI_REQUIRE(n_ranges >= 1 && n_ranges <= 64 && (n_ranges == 1 || (workspace && n_tokens <= 65535)), "gated_attention_mma: key ranges need a workspace (1 to 64 ranges, at most 65535 tokens)");
     QI_REQUIRE(qi_gated_attention_mma_supported(nq, nkv, d, dv), "gated_attention_mma: heads %d/%d of %d/%d are not covered", nq, nkv, d, dv);
     QI_REQUIRE(n_entries >= 0 && n_tokens >= 0 && page_size > 0 && max_blocks > 0 && num_pages > 0, "gated_attention_mma: bad sizes");
@@ -369,7 +396,7 @@ extern "C" int qi_gated_attention_mma_ranges(const void* q, void* out, const voi
     const float sl = scale * 1.4426950408889634f;
 #define QI_GA(DKP, DVP)                                                                                                      \
     return launch_one<DKP, DVP>(grid, stream, q, out, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, q_start, \
-                                start_pos, n_entries, nq, nkv, d, dv, sl, softcap, out_scale, window, chunk, gate, ldg, sink, n_ranges, ws_o, ws_ml, n_tokens, status)
+                                start_pos, n_entries, nq, nkv, d, dv, sl, softcap, out_scale, window, chunk, gate, ldg, sink, bias, bias_len, n_ranges, ws_o, ws_ml, n_tokens, status)
 #define QI_GA_ROW(DKP)                                   \
     switch (padded(dv)) {                                \
         case 32: QI_GA(DKP, 32);                         \
@@ -408,7 +435,7 @@ extern "C" int qi_gated_attention_mma_sink(const void* q, void* out, const void*
                                       int n_entries, int n_tokens, int nq, int nkv, int d, int dv, float scale, float softcap,
                                       float out_scale, int window, int chunk, const void* gate, long long ldg, const float* sink,
                                       int* status, cudaStream_t stream) {
-    return qi_gated_attention_mma_ranges(q, out, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, q_start, start_pos,
-                                         n_entries, n_tokens, nq, nkv, d, dv, scale, softcap, out_scale, window, chunk, gate, ldg, sink, 1,
+    return qi_gated_attention_mma_bias(q, out, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, q_start, start_pos,
+                                         n_entries, n_tokens, nq, nkv, d, dv, scale, softcap, out_scale, window, chunk, gate, ldg, sink, nullptr, 0, 1,
                                          nullptr, status, stream);
 }

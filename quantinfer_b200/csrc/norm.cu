@@ -10,10 +10,13 @@
 // reference's (backends/cpu/src/backend.rs:172-193: mean square :185-186,
 // inverse :187, scale :189; the residual add is crates/quantinfer-runtime/src/linear.rs:129-142).
 #include "common.cuh"
+#include "vec8.cuh"
 
 #include <cooperative_groups.h>
 
 namespace {
+
+using qi::Vec8;
 
 template <typename TD, typename TO>
 __global__ void add_rmsnorm_kernel(float* __restrict__ resid, const TD* __restrict__ delta,
@@ -51,37 +54,6 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ resid, const TD* __restri
 
 // The same, eight elements per thread and step (hidden a multiple of 8, rows 16-byte
 // aligned): 32-byte loads of the residual, 16-byte loads of a bfloat16 delta.
-template <typename T> struct Vec8;
-template <> struct Vec8<float> {
-    static __device__ __forceinline__ void load(const float* p, float (&v)[8]) {
-        const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-        v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-    }
-    static __device__ __forceinline__ void store(float* p, const float (&v)[8]) {
-        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-        *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
-    }
-};
-template <> struct Vec8<qi::bf16> {
-    static __device__ __forceinline__ void load(const qi::bf16* p, float (&v)[8]) {
-        const uint4 u = *reinterpret_cast<const uint4*>(p);
-        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const float2 f = __bfloat1622float2(h[i]);
-            v[2 * i] = f.x;
-            v[2 * i + 1] = f.y;
-        }
-    }
-    static __device__ __forceinline__ void store(qi::bf16* p, const float (&v)[8]) {
-        uint4 u;
-        __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&u);
-#pragma unroll
-        for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
-        *reinterpret_cast<uint4*>(p) = u;
-    }
-};
-
 QI_TL_DEFINE(qi_timeline_norm)
 
 template <typename TD, typename TO>

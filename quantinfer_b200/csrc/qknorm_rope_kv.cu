@@ -18,6 +18,7 @@
 // token at position p of request r lies in page table[r, p / page_size] at row
 // p % page_size.
 #include "common.cuh"
+#include "vec8.cuh"
 
 namespace {
 
@@ -300,9 +301,15 @@ extern "C" int qi_qk_norm_rope_kv(const void* qkv, int qkv_splits, void* q_out, 
 // head turn by angle = position * inv_freq[pair] (32-bit product, sincosf), pairs (i, i + rot / 2) or, when
 // `interleaved`, (2i, 2i + 1); q goes to q_out [n, nq d], k and v into the request's pages
 // (k_pages [pages, nkv, page_size, d], v_pages [pages, nkv, page_size, dv]; null: nothing is written).
-// Two options for designs that ask for them: one RMS norm over the whole of q and one over the whole of k (all heads
-// at once, gain per coordinate) before the rotation; and values that are the keys as projected (no v in the row).
+// Options for designs that ask for them: one RMS norm over the whole of q and one over the whole of k (all heads
+// at once, gain per coordinate) before the rotation, or one over every head by itself (`head_norm`; a gain of d numbers
+// that the heads share); values that are the keys as projected (no v in the row); and a factor on q that grows with the
+// position, 1 + temp_coef ln(floor((p + 1) / temp_every) + 1).
 namespace {
+
+__device__ __forceinline__ float query_factor(int pos, float temp_coef, int temp_every) {
+    return temp_every > 0 ? fmaf(temp_coef, logf((float)((pos + 1) / temp_every + 1)), 1.f) : 1.f;
+}
 
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -310,9 +317,10 @@ bias_rope_kv_kernel(const T* __restrict__ proj, long long ld, const float* __res
                     const float* __restrict__ inv_freq, int rot, int interleaved, const int* __restrict__ positions,
                     const int* __restrict__ token_req, const int* __restrict__ block_table, int max_blocks, int page_size,
                     int num_pages, T* __restrict__ k_pages, T* __restrict__ v_pages, int nq, int nkv, int d, int dv,
-                    const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps, int v_from_k,
-                    int* __restrict__ status) {
+                    const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps, int head_norm, int v_from_k,
+                    float temp_coef, int temp_every, int* __restrict__ status) {
     __shared__ float scratch[32];
+    extern __shared__ float head_inv[];         // [nq + nkv] with norms of every head by itself
     qi::pdl_wait();
     const int t = blockIdx.x;
     const int pos = positions[t];
@@ -324,7 +332,19 @@ bias_rope_kv_kernel(const T* __restrict__ proj, long long ld, const float* __res
     const int qk = (nq + nkv) * d, total = v_from_k ? qk : qk + nkv * dv;
     // one RMS norm over all of q and one over all of k (before the rotation), when their gains are given
     float q_inv = 1.f, k_inv = 1.f;
-    if (q_gain) {
+    if (q_gain && head_norm) {
+        const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+        for (int hd = warp; hd < nq + nkv; hd += blockDim.x >> 5) {
+            float sq = 0.f;
+            for (int i = lane; i < d; i += 32) {
+                const float x = qi::to_f32<T>(row[hd * d + i]) + (bias ? bias[hd * d + i] : 0.f);
+                sq = fmaf(x, x, sq);
+            }
+            sq = qi::warp_sum(sq);
+            if (lane == 0) head_inv[hd] = 1.0f / sqrtf(sq / (float)d + eps);
+        }
+        __syncthreads();
+    } else if (q_gain) {
         float sq = 0.f, sk = 0.f;
         for (int e = threadIdx.x; e < qk; e += blockDim.x) {
             const float x = qi::to_f32<T>(row[e]) + (bias ? bias[e] : 0.f);
@@ -335,7 +355,8 @@ bias_rope_kv_kernel(const T* __restrict__ proj, long long ld, const float* __res
     }
     auto normed = [&](int e) {
         float x = qi::to_f32<T>(row[e]) + (bias ? bias[e] : 0.f);
-        if (q_gain) x = e < nq * d ? x * q_inv * q_gain[e] : x * k_inv * k_gain[e - nq * d];
+        if (q_gain && head_norm) x = x * head_inv[e / d] * (e < nq * d ? q_gain : k_gain)[e % d];
+        else if (q_gain) x = e < nq * d ? x * q_inv * q_gain[e] : x * k_inv * k_gain[e - nq * d];
         return x;
     };
     T* krow = nullptr;
@@ -350,6 +371,7 @@ bias_rope_kv_kernel(const T* __restrict__ proj, long long ld, const float* __res
         }
     }
     const int half = rot / 2;
+    const float q_factor = query_factor(pos, temp_coef, temp_every);
     for (int e = threadIdx.x; e < total; e += blockDim.x) {
         if (e >= qk) {   // a value: bias only
             const int hv = (e - qk) / dv, i = (e - qk) % dv;
@@ -371,21 +393,79 @@ bias_rope_kv_kernel(const T* __restrict__ proj, long long ld, const float* __res
             sincosf((float)pos * inv_freq[pair], &sn, &cs);
             x = first ? x * cs - o * sn : x * cs + o * sn;
         }
-        if (head < nq) q_out[(size_t)t * nq * d + e] = qi::from_f32<T>(x);
+        if (head < nq) q_out[(size_t)t * nq * d + e] = qi::from_f32<T>(x * q_factor);
         else if (krow) krow[(size_t)(head - nq) * page_size * d + i] = qi::from_f32<T>(x);
+    }
+}
+
+// The form for rows without biases, rotation and values from keys, in 16-byte pieces: LANES lanes a head (eight coordinates
+// each, d <= 8 LANES), every operand read once. A warp takes 32 / LANES heads of q, k and v in turn.
+template <typename T, int LANES>
+__global__ void __launch_bounds__(256)
+head_norm_kv_kernel(const T* __restrict__ proj, long long ld, T* __restrict__ q_out, const int* __restrict__ positions,
+                    const int* __restrict__ token_req, const int* __restrict__ block_table, int max_blocks, int page_size,
+                    int num_pages, T* __restrict__ k_pages, T* __restrict__ v_pages, int nq, int nkv, int d, int dv,
+                    const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps, float temp_coef, int temp_every,
+                    int n_tokens, int* __restrict__ status) {
+    qi::pdl_wait();
+    const int heads = nq + 2 * nkv, per_block = 256 / LANES;
+    const int sub = threadIdx.x % LANES, i = sub * 8;
+    const long long total = (long long)n_tokens * heads;
+    for (long long it = (long long)blockIdx.x * per_block + threadIdx.x / LANES; it < (total + per_block - 1) / per_block * per_block;
+         it += (long long)gridDim.x * per_block) {
+        const bool in = it < total;           // whole warps stay together for the sums below
+        const int t = in ? (int)(it / heads) : 0, hd = in ? (int)(it % heads) : 0;
+        const bool is_v = hd >= nq + nkv;
+        const int width = is_v ? dv : d;
+        const T* src = proj + (size_t)t * ld + (is_v ? (size_t)(nq + nkv) * d + (size_t)(hd - nq - nkv) * dv : (size_t)hd * d);
+        float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+        if (in && i < width) qi::Vec8<T>::load(src + i, x);
+        float sq = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) sq = fmaf(x[j], x[j], sq);
+#pragma unroll
+        for (int o = LANES / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+        if (!in || i >= width) continue;      // nothing below is collective
+        const int pos = positions[t];
+        if (pos < 0) {
+            if (sub == 0 && status) atomicOr(status, qi::kStatusBadRange);
+            continue;
+        }
+        T* dst;
+        if (hd < nq) {
+            dst = q_out + ((size_t)t * nq + hd) * d;
+        } else {
+            if (!k_pages) continue;
+            const int page = block_table[(size_t)token_req[t] * max_blocks + pos / page_size];
+            if (page < 0 || page >= num_pages) {
+                if (sub == 0 && status) atomicOr(status, qi::kStatusBadPage);
+                continue;
+            }
+            const int g = is_v ? hd - nq - nkv : hd - nq;
+            dst = (is_v ? v_pages : k_pages) + (((size_t)page * nkv + g) * page_size + pos % page_size) * (size_t)width;
+        }
+        if (!is_v) {
+            float g[8];
+            qi::Vec8<float>::load((hd < nq ? q_gain : k_gain) + i, g);
+            const float inv = 1.0f / sqrtf(sq / (float)d + eps) * (hd < nq ? query_factor(pos, temp_coef, temp_every) : 1.f);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x[j] = x[j] * inv * g[j];
+        }
+        qi::Vec8<T>::store(dst + i, x);
     }
 }
 
 }  // namespace
 
 // q_gain, k_gain (both or neither; float32 [nq d], [nkv d]): q as a whole and k as a whole each pass an RMS norm with that
-// gain and `eps` before the rotation. v_from_k: the rows hold no v; a position's value is its key as projected (dv = d).
-extern "C" int qi_norm_rope_kv(const void* proj, long long ld, const float* bias, void* q_out, int dtype,
+// gain and `eps` before the rotation; with head_norm every head by itself does, with a gain of d numbers that the heads
+// share. temp_every > 0: q is multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1). v_from_k: the rows hold no v; a position's value is its key as projected (dv = d).
+extern "C" int qi_norm_rope_kv_ex(const void* proj, long long ld, const float* bias, void* q_out, int dtype,
                                const float* inv_freq, int rot, int interleaved, const int* positions,
                                const int* token_req, const int* block_table, int max_blocks, int page_size,
                                int num_pages, void* k_pages, void* v_pages, int n_tokens, int nq, int nkv, int d,
-                               int dv, const float* q_gain, const float* k_gain, float eps, int v_from_k, int* status,
-                               cudaStream_t stream) {
+                               int dv, const float* q_gain, const float* k_gain, float eps, int head_norm, int v_from_k, float temp_coef,
+                               int temp_every, int* status, cudaStream_t stream) {
     QI_REQUIRE(n_tokens >= 0 && nq > 0 && nkv > 0 && d > 0 && dv > 0, "bias_rope_kv: bad sizes");
     QI_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= d, "bias_rope_kv: %d rotated coordinates do not fit a head of %d", rot, d);
     QI_REQUIRE(rot == 0 || inv_freq, "bias_rope_kv: a rotation needs its inverse frequencies");
@@ -394,11 +474,31 @@ extern "C" int qi_norm_rope_kv(const void* proj, long long ld, const float* bias
     QI_REQUIRE(ld >= (long long)(nq + nkv) * d + (v_from_k ? 0 : (long long)nkv * dv), "bias_rope_kv: the rows are too short");
     QI_REQUIRE((k_pages == nullptr) == (v_pages == nullptr), "bias_rope_kv: key and value pages come together");
     QI_REQUIRE(!k_pages || (block_table && max_blocks > 0 && page_size > 0 && num_pages > 0), "bias_rope_kv: bad page geometry");
+    QI_REQUIRE(nq + nkv <= 8192, "bias_rope_kv: too many heads");
     if (n_tokens == 0) return 0;
+    if (q_gain && head_norm && !bias && !rot && !v_from_k && d % 8 == 0 && dv % 8 == 0 && d <= 256 && dv <= 256 && ld % 8 == 0 &&
+        (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)q_gain | (uintptr_t)k_gain) & 15) == 0) {
+        const int wide = d > dv ? d : dv;
+        const int lanes = wide <= 32 ? 4 : wide <= 64 ? 8 : wide <= 128 ? 16 : 32, per_block = 256 / lanes;
+        long long blocks = ((long long)n_tokens * (nq + 2 * nkv) + per_block - 1) / per_block;
+        if (blocks > 148 * 64) blocks = 148 * 64;
+#define QI_HN(L)                                                                                                                     \
+    qi::launch(head_norm_kv_kernel<T, L>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)proj, ld, (T*)q_out, positions, token_req, \
+               block_table, max_blocks, page_size, num_pages, (T*)k_pages, (T*)v_pages, nq, nkv, d, dv, q_gain, k_gain, eps, temp_coef, \
+               temp_every, n_tokens, status)
+        QI_DISPATCH_DTYPE(dtype, T, {
+            if (lanes == 4) QI_HN(4);
+            else if (lanes == 8) QI_HN(8);
+            else if (lanes == 16) QI_HN(16);
+            else QI_HN(32);
+        });
+#undef QI_HN
+        return qi::check_launch("head_norm_kv");
+    }
     QI_DISPATCH_DTYPE(dtype, T, {
-        qi::launch(bias_rope_kv_kernel<T>, dim3(n_tokens), dim3(256), 0, stream, (const T*)proj, ld, bias, (T*)q_out, inv_freq, rot,
+        qi::launch(bias_rope_kv_kernel<T>, dim3(n_tokens), dim3(256), head_norm ? sizeof(float) * (nq + nkv) : 0, stream, (const T*)proj, ld, bias, (T*)q_out, inv_freq, rot,
                    interleaved, positions, token_req, block_table, max_blocks, page_size, num_pages, (T*)k_pages, (T*)v_pages,
-                   nq, nkv, d, dv, q_gain, k_gain, eps, v_from_k, status);
+                   nq, nkv, d, dv, q_gain, k_gain, eps, head_norm, v_from_k, temp_coef, temp_every, status);
     });
     return qi::check_launch("bias_rope_kv");
 }
@@ -408,6 +508,6 @@ extern "C" int qi_bias_rope_kv(const void* proj, long long ld, const float* bias
                                const int* token_req, const int* block_table, int max_blocks, int page_size,
                                int num_pages, void* k_pages, void* v_pages, int n_tokens, int nq, int nkv, int d,
                                int dv, int* status, cudaStream_t stream) {
-    return qi_norm_rope_kv(proj, ld, bias, q_out, dtype, inv_freq, rot, interleaved, positions, token_req, block_table, max_blocks,
-                           page_size, num_pages, k_pages, v_pages, n_tokens, nq, nkv, d, dv, nullptr, nullptr, 0.f, 0, status, stream);
+    return qi_norm_rope_kv_ex(proj, ld, bias, q_out, dtype, inv_freq, rot, interleaved, positions, token_req, block_table, max_blocks,
+                           page_size, num_pages, k_pages, v_pages, n_tokens, nq, nkv, d, dv, nullptr, nullptr, 0.f, 0, 0, 0.f, 0, status, stream);
 }

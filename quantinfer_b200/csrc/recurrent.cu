@@ -1,7 +1,7 @@
 // Recurrent mixers whose state is of fixed size and 32-bit: a gated recurrence per channel (minGRU), and
 // recurrences over a matrix state per head that decays and receives the outer product k v^T of every token
 // (the time mixing of RWKV with a decay per key channel and a bonus for the current token; lightning
-// attention with one constant decay a head; the gated delta rule, whose state is decayed per key channel and corrected
+// attention with one constant decay a head; gated linear attention with a decay per key channel; the gated delta rule, whose state is decayed per key channel and corrected
 // towards each token's value). Beside them the small kernels these mixers need: the mix of a
 // token's input with its predecessor's (token shift) and the weighted sum of two branches' outputs.
 //
@@ -159,6 +159,8 @@ token_shift_kernel(const T* __restrict__ h, const float* __restrict__ mu, float*
 //   mode 0 (decay per key channel, bonus):   o_t = S_(t-1)^T r_t + (sum_i r_i u_i k_i) v_t ;  S_t = diag(w_t) S_(t-1) + k_t v_t^T
 //                                            w_t = exp(-exp(lw_t + w0)) from the decay projection's output lw
 //   mode 1 (one decay a head, silu inputs):  S_t = lambda S_(t-1) + k_t v_t^T ;  o_t = S_t^T q_t ;  q, k, v = silu of the projections
+//   mode 2 (decay per key channel, gated):   S_t = diag(w_t) S_(t-1) + k_t v_t^T ;  o_t = S_t^T (q_t q_scale) ;
+//                                            w_t = sigmoid(z_t + z0)^rate = exp(-rate softplus(-(z_t + z0))), z_t 32-bit
 // A block owns one entry, one head and up to kColThreads value columns; thread j keeps column j of S in registers
 // (DK numbers, dk padded with zeros). The operands of kStage tokens are staged in shared memory at a time (decays and
 // activations are evaluated there, once a token and channel: thread x stages key channels x, x + kColThreads, ...); in
@@ -172,14 +174,18 @@ token_shift_kernel(const T* __restrict__ h, const float* __restrict__ mu, float*
 
 constexpr int kColThreads = 64;
 
+// Type of the decay projection's output: mode 2 takes it in 32-bit.
+template <typename T, int MODE> struct DecayInput { typedef T type; };
+template <typename T> struct DecayInput<T, 2> { typedef float type; };
+
 template <typename T, int DK, int MODE>
 __global__ void __launch_bounds__(kColThreads, (DK <= 64 ? 8 : 1))
 matrix_state_scan_kernel(const T* __restrict__ r, long long ldr, const T* __restrict__ k, long long ldk, const T* __restrict__ v,
-                         long long ldv, const T* __restrict__ lw, long long ldw, const float* __restrict__ w0,
+                         long long ldv, const typename DecayInput<T, MODE>::type* __restrict__ lw, long long ldw, const float* __restrict__ w0,
                          const float* __restrict__ u, const float* __restrict__ lambda, float* __restrict__ state,
                          long long state_stride, float* __restrict__ o, float* __restrict__ decay_out, int write_state,
                          const int* __restrict__ q_start, const int* __restrict__ start_pos, const int* __restrict__ slot_ids,
-                         int heads, int dk, int dv) {
+                         int heads, int dk, int dv, float rate, float q_scale) {
     constexpr int kOwn = (DK + kColThreads - 1) / kColThreads;     // key channels a thread stages
     static_assert(DK % 4 == 0, "the staged operands are read four at a time");
     constexpr int kStage = DK <= 64 ? 8 : 4;                       // tokens a stage
@@ -215,14 +221,15 @@ matrix_state_scan_kernel(const T* __restrict__ r, long long ldr, const T* __rest
 #pragma unroll
     for (int m = 0; m < kOwn; ++m) {
         const int i = threadIdx.x + m * kColThreads;
-        const bool in = MODE == 0 && i < dk;
+        const bool in = MODE != 1 && i < dk;
         w0r[m] = in ? w0[(size_t)hd * dk + i] : 0.f;
         dsum[m] = 0.f;
     }
     if (MODE == 0)
         for (int i = threadIdx.x; i < DK; i += kColThreads) s_u[i] = i < dk ? u[(size_t)hd * dk + i] : 0.f;
     // A stage's numbers are fetched into registers one stage ahead, while the stage before is worked through.
-    T f_r[kOwn][kStage], f_k[kOwn][kStage], f_w[MODE == 0 ? kOwn : 1][kStage], f_v[kStage];
+    T f_r[kOwn][kStage], f_k[kOwn][kStage], f_v[kStage];
+    typename DecayInput<T, MODE>::type f_w[MODE != 1 ? kOwn : 1][kStage];
     auto fetch = [&](int base) {
         const int nt = min(kStage, len - base);
 #pragma unroll
@@ -235,7 +242,7 @@ matrix_state_scan_kernel(const T* __restrict__ r, long long ldr, const T* __rest
                     const size_t row = (size_t)(first + base + tt);
                     f_r[m][tt] = r[row * ldr + (size_t)hd * dk + i];
                     f_k[m][tt] = k[row * ldk + (size_t)hd * dk + i];
-                    if (MODE == 0) f_w[m][tt] = lw[row * ldw + (size_t)hd * dk + i];
+                    if (MODE != 1) f_w[m][tt] = lw[row * ldw + (size_t)hd * dk + i];
                 }
             }
         }
@@ -260,9 +267,15 @@ matrix_state_scan_kernel(const T* __restrict__ r, long long ldr, const T* __rest
                             rv = qi::to_f32<T>(f_r[m][tt]);
                             kv = qi::to_f32<T>(f_k[m][tt]);
                             if (MODE == 0) {
-                                const float rate = expf(qi::to_f32<T>(f_w[m][tt]) + w0r[m]);
-                                wv = expf(-rate);
-                                dsum[m] += rate;
+                                const float fall = expf(qi::to_f32<T>((T)f_w[m][tt]) + w0r[m]);
+                                wv = expf(-fall);
+                                dsum[m] += fall;
+                            } else if (MODE == 2) {
+                                const float z = (float)f_w[m][tt] + w0r[m];
+                                const float fall = rate * (log1pf(expf(-fabsf(z))) + fmaxf(-z, 0.f));   // rate softplus(-z)
+                                wv = expf(-fall);
+                                dsum[m] += fall;
+                                rv *= q_scale;
                             } else {
                                 rv = siluf_(rv);
                                 kv = siluf_(kv);
@@ -270,7 +283,7 @@ matrix_state_scan_kernel(const T* __restrict__ r, long long ldr, const T* __rest
                         }
                         s_r[tt][i] = rv;
                         s_k[tt][i] = kv;
-                        if (MODE == 0) s_w[tt][i] = wv;
+                        if (MODE != 1) s_w[tt][i] = wv;
                     }
                 }
             }
@@ -305,7 +318,7 @@ matrix_state_scan_kernel(const T* __restrict__ r, long long ldr, const T* __rest
 #pragma unroll
                 for (int i = 0; i < DK; i += 4) {
                     const float4 kk = k4[i >> 2];
-                    const float4 ww = MODE == 0 ? w4[i >> 2] : make_float4(lam, lam, lam, lam);
+                    const float4 ww = MODE != 1 ? w4[i >> 2] : make_float4(lam, lam, lam, lam);
                     S[i] = fmaf(ww.x, S[i], kk.x * vj);
                     S[i + 1] = fmaf(ww.y, S[i + 1], kk.y * vj);
                     S[i + 2] = fmaf(ww.z, S[i + 2], kk.z * vj);
@@ -337,13 +350,14 @@ matrix_state_scan_kernel(const T* __restrict__ r, long long ldr, const T* __rest
 #pragma unroll
                 for (int i = 0; i < DK; i += 4) {
                     const float4 rr = r4[i >> 2], kk = k4[i >> 2];
-                    S[i] = fmaf(lam, S[i], kk.x * vj);
+                    const float4 ww = MODE == 2 ? w4[i >> 2] : make_float4(lam, lam, lam, lam);
+                    S[i] = fmaf(ww.x, S[i], kk.x * vj);
                     acc4[0] = fmaf(rr.x, S[i], acc4[0]);
-                    S[i + 1] = fmaf(lam, S[i + 1], kk.y * vj);
+                    S[i + 1] = fmaf(ww.y, S[i + 1], kk.y * vj);
                     acc4[1] = fmaf(rr.y, S[i + 1], acc4[1]);
-                    S[i + 2] = fmaf(lam, S[i + 2], kk.z * vj);
+                    S[i + 2] = fmaf(ww.z, S[i + 2], kk.z * vj);
                     acc4[2] = fmaf(rr.z, S[i + 2], acc4[2]);
-                    S[i + 3] = fmaf(lam, S[i + 3], kk.w * vj);
+                    S[i + 3] = fmaf(ww.w, S[i + 3], kk.w * vj);
                     acc4[3] = fmaf(rr.w, S[i + 3], acc4[3]);
                 }
             }
@@ -368,7 +382,7 @@ matrix_state_scan_kernel(const T* __restrict__ r, long long ldr, const T* __rest
 #pragma unroll
         for (int m = 0; m < kOwn; ++m) {
             const int i = threadIdx.x + m * kColThreads;
-            if (i < dk) decay_out[((size_t)e * heads + hd) * dk + i] = MODE == 0 ? expf(-dsum[m]) : all;
+            if (i < dk) decay_out[((size_t)e * heads + hd) * dk + i] = MODE != 1 ? expf(-dsum[m]) : all;
         }
     }
 }
@@ -477,6 +491,8 @@ extern "C" int qi_matrix_state_scan_supported(int dk) { return dk > 0 && dk <= 2
 
 // mode 0: r, k, lw [n, >= heads dk], v [n, >= heads dv] in `dtype` (each with its own row stride); w0, u float32
 // [heads dk]; lambda unused. mode 1: r (the queries), k, v the same; lambda float32 [heads]; lw, w0, u unused.
+// mode 2: r (the queries), k, v the same; lw float32 [n, >= heads dk] whatever `dtype` is, w0 float32 [heads dk] (added to
+// it), `rate` the power of the sigmoid, `q_scale` a factor on the queries; u, lambda unused (as are rate and q_scale else).
 // state float32 [heads, dv, dk] a slot, `state_stride` floats apart; o float32 [n, heads dv], or null: no outputs
 // (a segment's own contribution is all that is wanted). decay_out (or null): float32 [n_entries, heads, dk], receives
 // the product of each entry's decays per key channel. write_state 0: the state is read, not written.
@@ -484,12 +500,13 @@ extern "C" int qi_matrix_state_scan(int mode, const void* r, long long ldr, cons
                                     const void* lw, long long ldw, int dtype, const float* w0, const float* u, const float* lambda,
                                     float* state, long long state_stride, float* o, float* decay_out, int write_state,
                                     const int* q_start, const int* start_pos, const int* slot_ids, int n_entries, int heads,
-                                    int dk, int dv, cudaStream_t stream) {
-    QI_REQUIRE(mode == 0 || mode == 1, "matrix_state_scan: unknown mode %d", mode);
+                                    int dk, int dv, float rate, float q_scale, cudaStream_t stream) {
+    QI_REQUIRE(mode >= 0 && mode <= 2, "matrix_state_scan: unknown mode %d", mode);
     QI_REQUIRE(n_entries >= 0 && heads > 0 && dv > 0 && qi_matrix_state_scan_supported(dk), "matrix_state_scan: bad sizes (keys of 1..256)");
     QI_REQUIRE(ldr >= (long long)heads * dk && ldk >= (long long)heads * dk && ldv >= (long long)heads * dv, "matrix_state_scan: the rows are too short");
-    QI_REQUIRE(mode == 1 || (lw && w0 && u && ldw >= (long long)heads * dk), "matrix_state_scan: the decay's operands are missing");
-    QI_REQUIRE(mode == 0 || lambda, "matrix_state_scan: the heads' decays are missing");
+    QI_REQUIRE(mode == 1 || (lw && w0 && (u || mode == 2) && ldw >= (long long)heads * dk), "matrix_state_scan: the decay's operands are missing");
+    QI_REQUIRE(mode != 2 || rate > 0.f, "matrix_state_scan: the sigmoid's power must be positive");
+    QI_REQUIRE(mode != 1 || lambda, "matrix_state_scan: the heads' decays are missing");
     QI_REQUIRE(state_stride >= (long long)heads * dk * dv, "matrix_state_scan: the slots of the state overlap");
     QI_REQUIRE(o || write_state, "matrix_state_scan: neither outputs nor the state are wanted");
     QI_REQUIRE(n_entries <= 65535 && (dv + kColThreads - 1) / kColThreads <= 65535, "matrix_state_scan: grid too large");
@@ -497,7 +514,7 @@ extern "C" int qi_matrix_state_scan(int mode, const void* r, long long ldr, cons
     const dim3 grid(heads, n_entries, (dv + kColThreads - 1) / kColThreads), block(kColThreads);
 #define QI_MS(DKP, MODE)                                                                                                        \
     qi::launch(matrix_state_scan_kernel<T, DKP, MODE>, grid, block, 0, stream, (const T*)r, ldr, (const T*)k, ldk, (const T*)v, ldv, \
-               (const T*)lw, ldw, w0, u, lambda, state, state_stride, o, decay_out, write_state, q_start, start_pos, slot_ids, heads, dk, dv)
+               (const typename DecayInput<T, MODE>::type*)lw, ldw, w0, u, lambda, state, state_stride, o, decay_out, write_state, q_start, start_pos, slot_ids, heads, dk, dv, rate, q_scale)
 #define QI_MS_DK(MODE)                              \
     if (dk <= 16) QI_MS(16, MODE);                  \
     else if (dk <= 32) QI_MS(32, MODE);             \
@@ -505,7 +522,7 @@ extern "C" int qi_matrix_state_scan(int mode, const void* r, long long ldr, cons
     else if (dk <= 128) QI_MS(128, MODE);           \
     else QI_MS(256, MODE)
     QI_DISPATCH_DTYPE(dtype, T, {
-        if (mode == 0) { QI_MS_DK(0); } else { QI_MS_DK(1); }
+        if (mode == 0) { QI_MS_DK(0); } else if (mode == 1) { QI_MS_DK(1); } else { QI_MS_DK(2); }
     });
 #undef QI_MS_DK
 #undef QI_MS
@@ -517,7 +534,7 @@ extern "C" int qi_matrix_state_scan(int mode, const void* r, long long ldr, cons
 // Blocks of the scan kernel (mode, key size, operand type) that one SM holds at a time, or 0 when it cannot be told:
 // whoever cuts long entries into segments sizes them so that the launch fills whole waves.
 extern "C" int qi_matrix_state_scan_blocks_per_sm(int mode, int dk, int dtype) {
-    if ((mode != 0 && mode != 1) || !qi_matrix_state_scan_supported(dk) || (dtype != qi::kF32 && dtype != qi::kBF16)) return 0;
+    if (mode < 0 || mode > 2 || !qi_matrix_state_scan_supported(dk) || (dtype != qi::kF32 && dtype != qi::kBF16)) return 0;
     int blocks = 0;
 #define QI_MS_OCC(DKP, MODE) cudaOccupancyMaxActiveBlocksPerMultiprocessor(&blocks, matrix_state_scan_kernel<T, DKP, MODE>, kColThreads, 0)
 #define QI_MS_OCC_DK(MODE)                          \
@@ -527,7 +544,7 @@ extern "C" int qi_matrix_state_scan_blocks_per_sm(int mode, int dk, int dtype) {
     else if (dk <= 128) QI_MS_OCC(128, MODE);       \
     else QI_MS_OCC(256, MODE)
     QI_DISPATCH_DTYPE(dtype, T, {
-        if (mode == 0) { QI_MS_OCC_DK(0); } else { QI_MS_OCC_DK(1); }
+        if (mode == 0) { QI_MS_OCC_DK(0); } else if (mode == 1) { QI_MS_OCC_DK(1); } else { QI_MS_OCC_DK(2); }
     });
 #undef QI_MS_OCC_DK
 #undef QI_MS_OCC

@@ -114,6 +114,8 @@ class Model:
                 return self.native.forward(batch)
         if self.embedding_state_entry is not None:
             resid = self.embedding(batch.token_ids, batch, self.embedding_view)
+        elif getattr(self.embedding, "wants_positions", False):
+            resid = self.embedding(batch.token_ids, batch.positions)
         else:
             resid = self.embedding(batch.token_ids)
         delta = None

@@ -25,7 +25,7 @@ STATUS_NON_FINITE = 4
 STATUS_WAIT_TIMEOUT = 8
 STATUS_BAD_RANGE = 16
 
-ABI_VERSION = 13
+ABI_VERSION = 14
 
 
 def status_names(code: int) -> list:
@@ -161,6 +161,21 @@ def embedding(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, status:
                                 table.shape[0], C.c_float(scale), _ptr(status), _stream())
 
 
+def embedding_sinusoid(table, ids, positions, freq, out, status, copies: int = 1, scale: float = 1.0) -> None:
+    """out[t, c, i] = table[ids[t], i] * scale + (sin for even i, cos for odd i)(positions[t] * freq[i // 2]) for every
+    copy c < `copies`. freq float64 [ceil(hidden / 2)]; out float32 [n, copies * hidden]."""
+    _req(table, "table", ndim=2)
+    _req(ids, "ids", torch.int32, 1)
+    _req(positions, "positions", torch.int32, 1)
+    _req(freq, "freq", torch.float64, 1)
+    _req(out, "out", torch.float32, 2)
+    n, hidden = ids.numel(), table.shape[1]
+    if positions.numel() != n or freq.numel() != (hidden + 1) // 2 or tuple(out.shape) != (n, copies * hidden):
+        raise KernelError("embedding_sinusoid: shapes do not agree")
+    _call("other", "embedding_sinusoid", library().qi_embedding_sinusoid, _ptr(table), _code(table), _ptr(ids), _ptr(positions),
+          _ptr(freq), _ptr(out), n, hidden, table.shape[0], int(copies), C.c_float(scale), _ptr(status), _stream())
+
+
 # --------------------------------------------------------------------------
 # norms
 
@@ -230,6 +245,54 @@ def add_layernorm(resid: torch.Tensor, delta, gain: torch.Tensor, bias, eps: flo
     _call('norm', "add_layernorm", library().qi_add_layernorm,
           _ptr(resid), _ptr(delta), _code(delta) if delta is not None else F32, splits, C.c_longlong(stride), _ptr(gain),
           _ptr(bias), C.c_float(eps), _ptr(out), _code(out), _ptr(rows), n_out, h, int(bool(write_resid)), _stream())
+
+
+def hyper_max_streams() -> int:
+    return int(library().qi_hyper_max_streams())
+
+
+def hyper_norm(streams, n_streams: int, y=None, mix=None, share=None, read=None, gain=None, bias=None, eps: float = 0.0,
+               center: bool = True, out=None, rows=None, write_back: bool = True) -> None:
+    """Between two sublayers of a model with residual streams: x_t <- sum_s mix[s, t] x_s + share[t] y (all streams at once,
+    y [n, w] or the partial sums [splits, n, w], None: the streams stay), u = sum_t read[t] x_t (read None: the plain
+    sum), out = norm(u) (layer norm with `center`, else RMS norm; gain float32 [w], bias float32 [w] or None; out None:
+    only the streams move on). streams float32 [n, n_streams * w], in place unless write_back is False or `rows` (int32,
+    source rows of out's rows) is given. mix float32 [n_streams, n_streams], share and read float32 [n_streams]."""
+    _req(streams, "streams", torch.float32, 2)
+    n = streams.shape[0]
+    if n_streams <= 0 or streams.shape[1] % n_streams:
+        raise KernelError(f"hyper_norm: rows of {streams.shape[1]} numbers are not {n_streams} streams")
+    w = streams.shape[1] // n_streams
+    splits, stride = 1, 0
+    if y is not None:
+        _req(y, "y")
+        if y.dim() == 3:
+            splits, stride = y.shape[0], y.shape[1] * y.shape[2]
+        if y.dim() not in (2, 3) or tuple(y.shape[-2:]) != (n, w):
+            raise KernelError(f"hyper_norm: y {tuple(y.shape)} does not match {n} rows of {w}")
+        _req(mix, "mix", torch.float32, 2)
+        _req(share, "share", torch.float32, 1)
+        if tuple(mix.shape) != (n_streams, n_streams) or share.numel() != n_streams:
+            raise KernelError("hyper_norm: mix and share do not fit the streams")
+    if read is not None:
+        _req(read, "read", torch.float32, 1)
+        if read.numel() != n_streams:
+            raise KernelError("hyper_norm: one weight a stream")
+    n_out = n
+    if rows is not None:
+        _req(rows, "rows", torch.int32, 1)
+        n_out, write_back = rows.numel(), False
+    if out is not None:
+        _req(out, "out", ndim=2)
+        _req(gain, "gain", torch.float32, 1)
+        if bias is not None:
+            _req(bias, "bias", torch.float32, 1)
+        if tuple(out.shape) != (n_out, w) or gain.numel() != w or (bias is not None and bias.numel() != w):
+            raise KernelError(f"hyper_norm: out {tuple(out.shape)} / gain do not match {n_out} rows of {w}")
+    _call("norm", "hyper_norm", library().qi_hyper_norm, _ptr(streams), _ptr(y), _code(y) if y is not None else F32, splits,
+          C.c_longlong(stride), _ptr(mix if y is not None else None), _ptr(share if y is not None else None), _ptr(read), _ptr(gain),
+          _ptr(bias), C.c_float(eps), int(bool(center)), _ptr(out), _code(out) if out is not None else F32, _ptr(rows), n_out,
+          n_streams, w, int(bool(write_back)), _stream())
 
 
 def scale_add_rmsnorm(resid: torch.Tensor, delta, alpha: float, gain: torch.Tensor, eps: float, copy=None) -> None:
@@ -387,15 +450,25 @@ def qk_norm_rope_kv(qkv, q_out, q_gain, k_gain, eps, cos, sin, rotary_dim, posit
 # attention
 
 
+def _req_bias(bias, nq: int) -> None:
+    """A distance bias of the attention kernels: float32 [nq, reach], reach >= 1."""
+    if bias is not None:
+        _req(bias, "bias", torch.float32, 2)
+        if bias.shape[0] != nq or bias.shape[1] < 1:
+            raise KernelError(f"attention: a distance bias of shape {tuple(bias.shape)} for {nq} query heads")
+
+
 def attention_generic(q, out, k_pages, v_pages, block_table, positions, token_req, nq, nkv, d,
                       scale: float, window: int, status, chunk: int = 0, gate=None, softcap: float = 0.0,
-                      out_scale: float = 1.0, sink=None) -> None:
+                      out_scale: float = 1.0, sink=None, bias=None) -> None:
     """Causal paged GQA attention, 32-bit arithmetic, any span length and page size. `sink` (float32 [nq] or None): the
     softmax's denominator of head h holds exp(sink[h]) once more, with no key and no value. Values may have another
     size than keys (v_pages [pages, nkv, page_size, dv], out [n, nq dv]); `chunk` > 0: a query sees only the keys
     of its own chunk of that many positions (counted from the sequence's start); `gate` [n, >= nq dv] (a view whose
     rows may lie further apart): the result is multiplied by sigmoid(gate). `softcap` c > 0: a score s becomes
-    c tanh(s / c) before the softmax. `out_scale` multiplies the result."""
+    c tanh(s / c) before the softmax. `out_scale` multiplies the result. `bias` (float32 [nq, reach] or None): a key n
+    positions back adds bias[h, min(n, reach - 1)] to its score (after the cap)."""
+    _req_bias(bias, nq)
     _req(q, "q", ndim=2)
     _req(out, "out", q.dtype, 2)
     _req(k_pages, "k_pages", q.dtype, 4)
@@ -418,10 +491,11 @@ def attention_generic(q, out, k_pages, v_pages, block_table, positions, token_re
         _req(sink, "sink", torch.float32, 1)
         if sink.numel() != nq:
             raise KernelError("attention: one sink a query head")
-    _call('attention', "attention_generic", library().qi_attention_generic_sink,
+    _call('attention', "attention_generic", library().qi_attention_generic_bias,
           _ptr(q), _ptr(out), _code(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
         block_table.shape[1], k_pages.shape[2], k_pages.shape[0], _ptr(positions), _ptr(token_req), n,
-        nq, nkv, d, dv, C.c_float(scale), C.c_float(softcap or 0.0), C.c_float(out_scale), int(window or 0), int(chunk or 0), _ptr(gate), C.c_longlong(ldg), _ptr(sink), _ptr(status), _stream())
+        nq, nkv, d, dv, C.c_float(scale), C.c_float(softcap or 0.0), C.c_float(out_scale), int(window or 0), int(chunk or 0), _ptr(gate), C.c_longlong(ldg), _ptr(sink),
+        _ptr(bias), bias.shape[1] if bias is not None else 0, _ptr(status), _stream())
 
 
 def attention_mma_supported(nq: int, nkv: int, d: int) -> bool:
@@ -469,7 +543,7 @@ def attention_prefill_ranges(n_ctas: int, max_kv_len: int) -> int:
 def attention_prefill(q, out, k_pages, v_pages, block_table, q_start, start_pos, tile_req, tile_q0,
                       nq, nkv, d, scale: float, window: int, status, use_tma: bool | None = None,
                       impl: str | None = None, max_kv_len: int = 0, key_ranges: int | None = None, chunk: int = 0,
-                      gate=None, softcap: float = 0.0, out_scale: float = 1.0, sink=None) -> None:
+                      gate=None, softcap: float = 0.0, out_scale: float = 1.0, sink=None, bias=None) -> None:
     """Causal paged GQA flash attention (bfloat16, head size 64 or 128) for spans of any
     length. `tile_req[i]`, `tile_q0[i]`: request index and first flat token of the i-th
     block of up to QUERY_TILE query rows.
@@ -483,7 +557,9 @@ def attention_prefill(q, out, k_pages, v_pages, block_table, q_start, start_pos,
     `chunk` (a query sees only the keys of its own chunk of that many positions, counted from the sequence's
     start), `gate` (bfloat16 [n, nq d], rows a multiple of 8 elements apart and 16-byte aligned: the output is
     multiplied with its sigmoid), `softcap` c > 0 (a score s becomes c tanh(s / c)), `out_scale` (a factor on the
-    result) and `sink` (float32 [nq]: exp(sink[h]) once more in the softmax's denominator of head h)."""
+    result), `sink` (float32 [nq]: exp(sink[h]) once more in the softmax's denominator of head h) and `bias` (float32
+    [nq, reach]: a key n positions back adds bias[h, min(n, reach - 1)] to its score)."""
+    _req_bias(bias, nq)
     if impl is None and use_tma is not None:
         impl = "tma" if use_tma else "cpasync"
     _req(q, "q", torch.bfloat16, 2)
@@ -518,14 +594,15 @@ def attention_prefill(q, out, k_pages, v_pages, block_table, q_start, start_pos,
             ldg = gate.stride(0)
         if sink is not None:
             _req(sink, "sink", torch.float32, 1)
-        _call('attention', "attention_prefill_tcgen05", library().qi_attention_prefill_tcgen05_sink,
+        _call('attention', "attention_prefill_tcgen05", library().qi_attention_prefill_tcgen05_bias,
               _ptr(q), _ptr(out), _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],
             k_pages.shape[2], k_pages.shape[0], _ptr(q_start), _ptr(start_pos), _ptr(tile_req), _ptr(tile_q0),
             tile_req.numel(), q.shape[0], nq, nkv, d, C.c_float(scale), int(window or 0), int(chunk or 0), _ptr(gate),
-            C.c_longlong(ldg), ranges, _ptr(ws), _ptr(status), C.c_float(softcap or 0.0), C.c_float(out_scale), _ptr(sink), _stream())
+            C.c_longlong(ldg), ranges, _ptr(ws), _ptr(status), C.c_float(softcap or 0.0), C.c_float(out_scale), _ptr(sink),
+            _ptr(bias), bias.shape[1] if bias is not None else 0, _stream())
         return
-    if chunk or gate is not None or softcap or out_scale != 1.0 or sink is not None:
-        raise KernelError(f"attention_prefill: the {impl!r} kernel takes neither a chunk bound, a gate, a soft cap, an output factor nor a sink")
+    if chunk or gate is not None or softcap or out_scale != 1.0 or sink is not None or bias is not None:
+        raise KernelError(f"attention_prefill: the {impl!r} kernel takes neither a chunk bound, a gate, a soft cap, an output factor, a sink nor a bias")
     if impl not in ("tma", "cpasync"):
         raise KernelError(f"attention_prefill: unknown kernel {impl!r}")
     if impl == "tma":
@@ -1174,13 +1251,15 @@ def concat_cast(a, b, out) -> None:
 
 def bias_rope_kv(proj, bias, q_out, inv_freq, rot: int, interleaved: bool, positions, token_req, block_table, page_size: int,
                  k_pages, v_pages, nq: int, nkv: int, d: int, dv: int, status, q_gain=None, k_gain=None, norm_eps: float = 0.0,
-                 values_from_keys: bool = False) -> None:
+                 values_from_keys: bool = False, head_norm: bool = False, q_temp=None) -> None:
     """proj [n, >= (nq + nkv) d + nkv dv] holds q | k | v (more columns may follow); bias float32 over those columns or
     None; the first `rot` coordinates of each q and k head turn by position * inv_freq[pair] (computed here in 32-bit:
     no table, no limit on positions); q goes to q_out [n, nq d], k and v into the pages (None: nothing is written).
     q_gain, k_gain (float32 [nq d], [nkv d]; both or neither): all of q and all of k each pass one RMS norm with that gain
     and `norm_eps` before the rotation. values_from_keys: the rows hold no v; a position's value is its key as
-    projected, before norm and rotation (dv = d)."""
+    projected, before norm and rotation (dv = d). head_norm: every head of q and k passes an RMS norm of its own instead, with
+    gains q_gain, k_gain [d] that the heads share. q_temp (coef, every) or None: q is multiplied by
+    1 + coef ln(floor((p + 1) / every) + 1) at position p."""
     if not proj.is_cuda or proj.dim() != 2 or proj.stride(1) != 1:
         raise KernelError("bias_rope_kv: proj must be a CUDA tensor with contiguous rows")
     _req(q_out, "q_out", proj.dtype, 2)
@@ -1191,7 +1270,7 @@ def bias_rope_kv(proj, bias, q_out, inv_freq, rot: int, interleaved: bool, posit
     if q_gain is not None:
         _req(q_gain, "q_gain", torch.float32, 1)
         _req(k_gain, "k_gain", torch.float32, 1)
-        if q_gain.numel() != nq * d or k_gain.numel() != nkv * d:
+        if q_gain.numel() != (d if head_norm else nq * d) or k_gain.numel() != (d if head_norm else nkv * d):
             raise KernelError("bias_rope_kv: the gains do not fit q and k")
     if proj.shape[1] < cols or tuple(q_out.shape) != (n, nq * d):
         raise KernelError(f"bias_rope_kv: proj {tuple(proj.shape)} / q_out {tuple(q_out.shape)} do not match the heads")
@@ -1213,10 +1292,11 @@ def bias_rope_kv(proj, bias, q_out, inv_freq, rot: int, interleaved: bool, posit
         if tuple(k_pages.shape[1:]) != (nkv, page_size, d) or tuple(v_pages.shape) != (k_pages.shape[0], nkv, page_size, dv):
             raise KernelError(f"bias_rope_kv: pages {tuple(k_pages.shape)} / {tuple(v_pages.shape)} do not fit")
         num_pages, max_blocks = k_pages.shape[0], block_table.shape[1]
-    _call("rope", "bias_rope_kv", library().qi_norm_rope_kv, _ptr(proj), C.c_longlong(proj.stride(0)), _ptr(bias), _ptr(q_out),
+    _call("rope", "bias_rope_kv", library().qi_norm_rope_kv_ex, _ptr(proj), C.c_longlong(proj.stride(0)), _ptr(bias), _ptr(q_out),
           _code(proj), _ptr(inv_freq if rot else None), rot, int(bool(interleaved)), _ptr(positions), _ptr(token_req),
           _ptr(block_table), max_blocks, page_size, num_pages, _ptr(k_pages), _ptr(v_pages), n, nq, nkv, d, dv, _ptr(q_gain),
-          _ptr(k_gain), C.c_float(norm_eps), int(bool(values_from_keys)), _ptr(status), _stream())
+          _ptr(k_gain), C.c_float(norm_eps), int(bool(head_norm)), int(bool(values_from_keys)), C.c_float(q_temp[0] if q_temp else 0.0),
+          int(q_temp[1]) if q_temp else 0, _ptr(status), _stream())
 
 
 def ssm_scan(xbc, raw_dt, dt_bias, a_log, d_skip, state, y, q_start, start_pos, slot_ids, heads: int, groups: int, P: int, N: int,
@@ -1342,13 +1422,19 @@ def token_shift(h, mu, state, out, token_req, q_start, start_pos, slot_ids) -> N
           _ptr(out), _ptr(token_req), _ptr(q_start), _ptr(start_pos), _ptr(slot_ids), n, ch, mu.shape[0], _stream())
 
 
+SCAN_MODES = {"channel_decay": 0, "head_decay": 1, "channel_gate": 2}
+
+
 def matrix_state_scan(mode: str, r, k, v, state, o, q_start, start_pos, slot_ids, heads: int, dk: int, dv: int, *, log_decay=None,
                       decay_bias=None, bonus=None, head_decay=None, decay_out=None, write_state: bool = True, beta=None,
-                      qk_heads: int | None = None, unit_eps: float = 1e-6, q_scale: float = 1.0, prepared: bool | None = None) -> None:
+                      qk_heads: int | None = None, unit_eps: float = 1e-6, q_scale: float = 1.0, prepared: bool | None = None,
+                      rate: float = 1.0) -> None:
     """A recurrence over a matrix state S [dk, dv] a head that decays and receives k_t v_t^T with every token.
     mode "channel_decay": o_t = S_(t-1)^T r_t + (sum_i r_i bonus_i k_i) v_t, then S_t = diag(w_t) S_(t-1) + k_t v_t^T with
     w_t = exp(-exp(log_decay_t + decay_bias)) per head and key channel. mode "head_decay": r, k, v pass silu first,
-    S_t = head_decay S_(t-1) + k_t v_t^T, o_t = S_t^T r_t. r, k, log_decay [n, heads dk], v [n, heads dv] (blocks of
+    S_t = head_decay S_(t-1) + k_t v_t^T, o_t = S_t^T r_t. mode "channel_gate": S_t = diag(w_t) S_(t-1) + k_t v_t^T,
+    o_t = S_t^T (r_t q_scale), w_t = sigmoid(log_decay_t + decay_bias)^rate per head and key channel, with log_decay (the
+    gate's logits) float32 whatever the type of r. r, k, log_decay [n, heads dk], v [n, heads dv] (blocks of
     columns of wider rows are fine); decay_bias, bonus float32 [heads dk]; head_decay float32 [heads]; state float32
     [slots, heads, dv, dk]; o float32 [n, heads dv], or None: the state moves on and nothing else is written. decay_out
     (or None): float32 [entries, heads, dk], receives the product of each entry's decays per key channel. write_state
@@ -1362,7 +1448,7 @@ def matrix_state_scan(mode: str, r, k, v, state, o, q_start, start_pos, slot_ids
     state to the next, and a prompt of one request spreads over heads x (dv / columns a block) blocks. `prepared`: True
     runs the two-launch form (unit vectors, decays and beta once a token, then a scan fed by asynchronous copies), False
     the one-launch form; None: the two-launch form for steps of more than four tokens an entry."""
-    if mode not in ("channel_decay", "head_decay", "delta"):
+    if mode not in SCAN_MODES and mode != "delta":
         raise KernelError(f"matrix_state_scan: unknown mode {mode!r}")
     for t, name in ((r, "r"), (k, "k"), (v, "v")):
         _cols(t, name, r.dtype)
@@ -1380,6 +1466,11 @@ def matrix_state_scan(mode: str, r, k, v, state, o, q_start, start_pos, slot_ids
         if tuple(log_decay.shape) != (n, heads * dk) or tuple(beta.shape) != (n, heads) or decay_bias.numel() != heads * dk or (
                 head_decay.numel() != heads) or decay_out is not None:
             raise KernelError("matrix_state_scan: the delta rule's operands do not fit the heads")
+    elif mode == "channel_gate":
+        _cols(log_decay, "log_decay", torch.float32)
+        _req(decay_bias, "decay_bias", torch.float32)
+        if log_decay.shape != r.shape or decay_bias.numel() != heads * dk or rate <= 0.0:
+            raise KernelError("matrix_state_scan: the decay's operands do not fit the heads")
     elif channel:
         _cols(log_decay, "log_decay", r.dtype)
         _req(decay_bias, "decay_bias", torch.float32)
@@ -1417,11 +1508,11 @@ def matrix_state_scan(mode: str, r, k, v, state, o, q_start, start_pos, slot_ids
               _ptr(q_start), _ptr(start_pos), _ptr(slot_ids), start_pos.numel(), heads, qk_heads, dk, dv, C.c_float(unit_eps),
               C.c_float(q_scale), _ptr(scratch), n, _stream())
         return
-    _call("scan", "matrix_state_scan", library().qi_matrix_state_scan, 0 if channel else 1, _ptr(r), C.c_longlong(r.stride(0)), _ptr(k),
-          C.c_longlong(k.stride(0)), _ptr(v), C.c_longlong(v.stride(0)), _ptr(log_decay), C.c_longlong(log_decay.stride(0) if channel else 0),
+    _call("scan", "matrix_state_scan", library().qi_matrix_state_scan, SCAN_MODES[mode], _ptr(r), C.c_longlong(r.stride(0)), _ptr(k),
+          C.c_longlong(k.stride(0)), _ptr(v), C.c_longlong(v.stride(0)), _ptr(log_decay), C.c_longlong(log_decay.stride(0) if log_decay is not None else 0),
           _code(r), _ptr(decay_bias), _ptr(bonus), _ptr(head_decay), _ptr(state), C.c_longlong(state.stride(0)), _ptr(o),
           _ptr(decay_out), int(bool(write_state)), _ptr(q_start), _ptr(start_pos), _ptr(slot_ids), start_pos.numel(), heads, dk, dv,
-          _stream())
+          C.c_float(rate), C.c_float(q_scale), _stream())
 
 
 def matrix_state_chain(seg_state, seg_decay, state, entry_seg, start_pos, slot_ids) -> None:
@@ -1467,7 +1558,7 @@ def matrix_state_scan_blocks(mode: str, dk: int, dtype) -> int:
     cannot be told. For whoever cuts long entries into segments: a launch of whole waves wastes no time on a tail."""
     key = (mode, dk, dtype)
     if key not in _SCAN_BLOCKS:
-        a_sm = int(library().qi_matrix_state_scan_blocks_per_sm(0 if mode == "channel_decay" else 1, int(dk), _DTYPE_CODE[dtype]))
+        a_sm = int(library().qi_matrix_state_scan_blocks_per_sm(SCAN_MODES[mode], int(dk), _DTYPE_CODE[dtype]))
         _SCAN_BLOCKS[key] = max(0, a_sm) * torch.cuda.get_device_properties(torch.cuda.current_device()).multi_processor_count
     return _SCAN_BLOCKS[key]
 
@@ -1589,14 +1680,15 @@ def gated_attention_mma_supported(nq: int, nkv: int, d: int, dv: int) -> bool:
 
 def gated_attention(q, out, k_pages, v_pages, block_table, batch, nq, nkv, d, dv, scale: float, window: int, chunk: int, gate,
                     status, impl: str | None = None, softcap: float = 0.0, out_scale: float = 1.0, sink=None,
-                    key_ranges: int | None = None) -> None:
+                    key_ranges: int | None = None, bias=None) -> None:
     """Attention with separate key and value sizes, an optional chunk bound and an optional output gate, by the
     kernel that fits: "mma" (bfloat16, head sizes that are multiples of 8 up to 128: flash form on the tensor
     cores, tiles found on the device from the step's arrays) or "generic" (32-bit arithmetic, any sizes). A step
     with prompt portions whose keys and values are both of size 128 goes to "tcgen05": the portions' query tiles
     to the tcgen05 flash kernel (chunk bound and gate included), the single tokens in front of them to "mma".
     `softcap` c > 0 (a score s becomes c tanh(s / c)), `out_scale` (a factor on the result) and `sink` (float32 [nq]:
-    exp(sink[h]) once more in the softmax's denominator of head h) are known to all three. A step of single tokens on
+    exp(sink[h]) once more in the softmax's denominator of head h) are known to all three, and so is `bias` (float32
+    [nq, reach]: a key n positions back adds bias[h, min(n, reach - 1)] to its score). A step of single tokens on
     "mma" cuts every token's keys into `key_ranges` ranges over separate CTAs (None: as many as fill the device, from
     the longest context and the window, so that a captured step serves its whole context bucket) and adds the parts
     in a second kernel."""
@@ -1609,17 +1701,18 @@ def gated_attention(q, out, k_pages, v_pages, block_table, batch, nq, nkv, d, dv
         if lead:
             gated_attention(q[:lead], out[:lead], k_pages, v_pages, block_table[:lead], _LeadRows(batch, lead), nq, nkv, d, dv,
                             scale, window, chunk, gate[:lead] if gate is not None else None, status, impl="mma", softcap=softcap,
-                            out_scale=out_scale, sink=sink)
+                            out_scale=out_scale, sink=sink, bias=bias)
         return attention_prefill(q, out, k_pages, v_pages, block_table, batch.q_start, batch.start_pos, batch.tile_req,
                                  batch.tile_q0, nq, nkv, d, scale, window, status, impl="tcgen05", max_kv_len=batch.max_kv_len,
                                  key_ranges=1 if chunk else None, chunk=chunk, gate=gate, softcap=softcap, out_scale=out_scale,
-                                 sink=sink)
+                                 sink=sink, bias=bias)
     if impl is None:
         impl = "mma" if q.dtype == torch.bfloat16 and gated_attention_mma_supported(nq, nkv, d, dv) and (
             gate is None or gate.stride(0) % 2 == 0) else "generic"
     if impl == "generic":
         return attention_generic(q, out, k_pages, v_pages, block_table, batch.positions, batch.token_req, nq, nkv, d, scale,
-                                 window, status, chunk=chunk, gate=gate, softcap=softcap, out_scale=out_scale, sink=sink)
+                                 window, status, chunk=chunk, gate=gate, softcap=softcap, out_scale=out_scale, sink=sink, bias=bias)
+    _req_bias(bias, nq)
     if sink is not None:
         _req(sink, "sink", torch.float32, 1)
         if sink.numel() != nq:
@@ -1645,8 +1738,9 @@ def gated_attention(q, out, k_pages, v_pages, block_table, batch, nq, nkv, d, dv
         ranges = key_ranges or max(1, min(-(-keys // 128), 296 // max(n * nq, 1), 64))
         if ranges > 1:
             ws = torch.empty(n * nq * ranges * (dv + 2), dtype=torch.float32, device=q.device)
-    _call("attention", "gated_attention_mma", library().qi_gated_attention_mma_ranges, _ptr(q), _ptr(out), _ptr(k_pages), _ptr(v_pages),
+    _call("attention", "gated_attention_mma", library().qi_gated_attention_mma_bias, _ptr(q), _ptr(out), _ptr(k_pages), _ptr(v_pages),
           _ptr(block_table), block_table.shape[1], k_pages.shape[2], k_pages.shape[0], _ptr(batch.q_start), _ptr(batch.start_pos),
           batch.n_requests, n, nq, nkv, d, dv, C.c_float(scale), C.c_float(softcap or 0.0), C.c_float(out_scale), int(window or 0),
-          int(chunk or 0), _ptr(gate), C.c_longlong(ldg), _ptr(sink), ranges, _ptr(ws),
+          int(chunk or 0), _ptr(gate), C.c_longlong(ldg), _ptr(sink),
+          _ptr(bias), bias.shape[1] if bias is not None else 0, ranges, _ptr(ws),
           _ptr(status), _stream())

@@ -309,6 +309,69 @@ class PostNormBlock(Part):
         return resid, StreamCopy(x)
 
 
+class HyperBlock(Part):
+    """A block over residual streams x_1 .. x_s (hyper-connections), kept side by side in a token's row of `resid`. For the
+    mixer, then the feed-forward (which may be absent):
+
+        u = sum_s in[s] x_s ;  y = sublayer(norm(u)) ;  x_t <- sum_s mix[s, t] x_s + out[t] y      (all streams at once)
+
+    The streams receive y in the kernel that reads them next (`read_streams`, in this block, the next one or the final
+    norm): what a block hands on is a :class:`StreamsPending`, y with the sublayer's mix and shares."""
+
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        if not 1 <= spec.streams <= 16:
+            raise ConfigError(f"hyper: {spec.streams} residual streams (1..16)")
+        if len(spec.names) != (2 if spec.ffn is not None else 1):
+            raise ConfigError("hyper: one name of connection tensors a sublayer")
+        self.mixer_norm = build_part("norm", spec.mixer_norm, runtime)
+        self.mixer = build_part("mixer", spec.mixer, runtime)
+        self.ffn = build_part("ffn", spec.ffn, runtime) if spec.ffn is not None else None
+        self.ffn_norm = build_part("norm", spec.ffn_norm, runtime) if spec.ffn is not None else None
+        if hasattr(self.mixer, "keep_partials"):
+            self.mixer.keep_partials = True       # the streams' kernel adds a split product's partial sums itself
+        self.read, self.share, self.mix = [], [], []
+        self._parts = tuple(p for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn) if p is not None)
+
+    @classmethod
+    def needs_of_spec(cls, spec):
+        needs = {}
+        subs = [("norm", spec.mixer_norm), ("mixer", spec.mixer)]
+        if spec.ffn is not None:
+            subs += [("norm", spec.ffn_norm), ("ffn", spec.ffn)]
+        for cat, sub in subs:
+            needs.update(part_class(cat, sub).needs_of_spec(sub))
+        s = spec.streams
+        for name in spec.names:
+            needs.update({name + ".in": TensorNeed((s,), "gain", "gain"), name + ".out": TensorNeed((s,), "gain", "gain"),
+                          name + ".mix": TensorNeed((s, s), "gain", "identity")})
+        return needs
+
+    def load(self, tensors):
+        for p in self._parts:
+            p.load(tensors)
+        names = self.spec.names
+        self.read, self.share, self.mix = ([self._gain(tensors[n + tail]) for n in names] for tail in (".in", ".out", ".mix"))
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def mixer_state_need(self):
+        return getattr(self.mixer, "state_need", lambda: None)()
+
+    def forward(self, resid, delta, batch, cache):
+        from .norm import StreamsPending, read_streams
+
+        s = self.spec.streams
+        h = read_streams(self.mixer_norm, resid, delta, s, self.read[0])
+        delta = StreamsPending(self.mixer.forward(h, batch, cache), self.mix[0], self.share[0])
+        if self.ffn is not None:
+            h = read_streams(self.ffn_norm, resid, delta, s, self.read[1])
+            delta = StreamsPending(self.ffn.forward(h), self.mix[1], self.share[1])
+        return resid, delta
+
+
+register_part("block", "hyper", HyperBlock)
 register_part("block", "postnorm", PostNormBlock)
 register_part("block", "prenorm", PreNormBlock)
 register_part("block", "sandwich", SandwichBlock)

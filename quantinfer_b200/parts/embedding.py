@@ -12,6 +12,7 @@ from __future__ import annotations
 import torch
 
 from .. import kernels
+from ..errors import ConfigError
 from ..weights.loader import TensorNeed
 from .base import Part, register_part
 from .linear import Linear
@@ -25,6 +26,14 @@ class Embedding(Part):
     def __init__(self, spec, runtime):
         super().__init__(spec, runtime)
         self.table = Linear(runtime, spec.vocab_size, spec.hidden_size, _weight_name(spec))
+        self.freq, self.copies = None, int(getattr(spec, "copies", 1))
+        base = getattr(spec, "sinusoid_base", None)
+        self.wants_positions = base is not None
+        if base is not None:        # angles are formed in 64-bit on the device
+            i = torch.arange((spec.hidden_size + 1) // 2, dtype=torch.float64)
+            self.freq = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / spec.hidden_size).to(runtime.device)
+        elif self.copies != 1:
+            raise ConfigError("embedding: copies for residual streams are written by the kernel with positions")
 
     @classmethod
     def needs_of_spec(cls, spec):
@@ -33,8 +42,13 @@ class Embedding(Part):
     def load(self, tensors):
         self.table.load(tensors[_weight_name(self.spec)])
 
-    def forward(self, token_ids):
-        out = torch.empty((token_ids.numel(), self.spec.hidden_size), dtype=torch.float32, device=token_ids.device)
+    def forward(self, token_ids, positions=None):
+        """The tokens' rows; with a position vector in the spec, `positions` (int32) says where the tokens stand."""
+        out = torch.empty((token_ids.numel(), self.copies * self.spec.hidden_size), dtype=torch.float32, device=token_ids.device)
+        if self.wants_positions:
+            kernels.embedding_sinusoid(self.table.weight, token_ids, positions, self.freq, out, self.runtime.status, self.copies,
+                                       getattr(self.spec, "scale", 1.0))
+            return out
         kernels.embedding(self.table.weight, token_ids, out, self.runtime.status, scale=getattr(self.spec, "scale", 1.0))
         return out
 

@@ -10,7 +10,9 @@
 Biases, the gate, the convolution, the cap and the factor are each optional (fields of the spec). So are: a sink (the
 softmax's denominator holds exp(b_h) once more, b zero or the learned tensor `sink`); one RMS norm over the whole of q
 and one over the whole of k before the rotation (`q.norm`, `k.norm`); values that are the keys as projected, before
-norm and rotation (no `v` then). The convolution's
+norm and rotation (no `v` then); or an RMS norm over every head of q and k by itself; a factor on q that grows with the
+position (`q_temp`); a learned number per head that a key's distance adds to its score (`distance_bias`, table `rel`,
+spread at load to one number a head and distance up to the first distance that reads the last row). The convolution's
 last taps - 1 projected rows are the mixer's state of fixed size BESIDE its pages (`state_need`, handed back as
 `cache.mixer_state`).
 
@@ -35,6 +37,7 @@ from ..errors import ConfigError
 from ..weights.loader import TensorNeed
 from .base import Part, register_part
 from .linear import Linear
+from .position import distance_buckets
 
 
 class GatedAttention(Part):
@@ -51,9 +54,12 @@ class GatedAttention(Part):
         self.sink_kind, self.qk_norm = getattr(s, "sink", None), getattr(s, "qk_norm", None)
         if self.v_from_k and (self.dv != self.d or getattr(s, "conv_taps", None) is not None or s.bias):
             raise ConfigError("gated_attention: values that are the keys have the keys' size, no bias and no convolution")
-        if self.sink_kind not in (None, "zero", "learned") or self.qk_norm not in (None, "whole"):
+        if self.sink_kind not in (None, "zero", "learned") or self.qk_norm not in (None, "whole", "head"):
             raise ConfigError(f"gated_attention: sink {self.sink_kind!r} / qk_norm {self.qk_norm!r} are not known")
-        self.sink = self.q_gain = self.k_gain = None
+        self.sink = self.q_gain = self.k_gain = self.dist_bias = None
+        self.q_temp, self.reach = getattr(s, "q_temp", None), getattr(s, "distance_bias", None)
+        if self.q_temp is not None and self.q_temp[1] < 1:
+            raise ConfigError("gated_attention: the query's factor grows every 1 or more positions")
         self.qkv_cols = (self.H + self.G) * self.d + (0 if self.v_from_k else self.G * self.dv)
         self.proj = Linear(runtime, self.qkv_cols + (self.H * self.dv if s.out_gate else 0), s.hidden_size, s.prefix + "q+k+v+g")
         if self.sink_kind == "zero":
@@ -80,6 +86,10 @@ class GatedAttention(Part):
             needs[p + "v"] = TensorNeed((G * dv, w))
         if getattr(s, "qk_norm", None) == "whole":
             needs.update({p + "q.norm": TensorNeed((H * d,), "gain", "gain"), p + "k.norm": TensorNeed((G * d,), "gain", "gain")})
+        if getattr(s, "qk_norm", None) == "head":
+            needs.update({p + "q.norm": TensorNeed((d,), "gain", "gain"), p + "k.norm": TensorNeed((d,), "gain", "gain")})
+        if getattr(s, "distance_bias", None) is not None:
+            needs[p + "rel"] = TensorNeed((None, H), "gain", "normal")
         if getattr(s, "sink", None) == "learned":
             needs[p + "sink"] = TensorNeed((H,), "gain", "normal")
         if s.out_gate:
@@ -96,8 +106,12 @@ class GatedAttention(Part):
     def load(self, tensors):
         p, s = self.spec.prefix, self.spec
         ws = [tensors[p + n] for n in ("q", "k") + (() if self.v_from_k else ("v",)) + (("g",) if s.out_gate else ())]
-        if self.qk_norm == "whole":
+        if self.qk_norm is not None:
             self.q_gain, self.k_gain = self._gain(tensors[p + "q.norm"]), self._gain(tensors[p + "k.norm"])
+        if self.reach is not None:
+            rel = tensors[p + "rel"].to(torch.float32)
+            buckets = distance_buckets(rel.shape[0], self.reach)
+            self.dist_bias = self._gain(rel[torch.tensor(buckets)].t())       # [heads, reach of the last row's edge + 1]
         if self.sink_kind == "learned":
             self.sink = self._gain(tensors[p + "sink"])
         if len({t.dtype for t in ws}) > 1:
@@ -137,12 +151,12 @@ class GatedAttention(Part):
                              table, cache.page_size, cache.k_pages if cache.writes else None,
                              cache.v_pages if cache.writes else None, self.H, self.G, self.d, self.dv, rt.status,
                              q_gain=self.q_gain, k_gain=self.k_gain, norm_eps=getattr(s, "qk_norm_eps", 0.0),
-                             values_from_keys=self.v_from_k)
+                             values_from_keys=self.v_from_k, head_norm=self.qk_norm == "head", q_temp=self.q_temp)
         out = torch.empty((n, self.H * self.dv), dtype=x.dtype, device=x.device)
         gate = gate_src[:, self.qkv_cols:] if s.out_gate else None
         kernels.gated_attention(q, out, cache.k_pages, cache.v_pages, table, batch, self.H, self.G, self.d, self.dv, s.scale,
                                 s.window or 0, s.chunk or 0, gate, rt.status, softcap=getattr(s, "softcap", None) or 0.0,
-                                out_scale=getattr(s, "out_scale", 1.0), sink=self.sink)
+                                out_scale=getattr(s, "out_scale", 1.0), sink=self.sink, bias=self.dist_bias)
         return self.o(out, keep_partials=True)
 
 

@@ -12,8 +12,9 @@ from __future__ import annotations
 import torch
 
 from .. import kernels
+from ..errors import ConfigError
 from ..weights.loader import TensorNeed
-from .base import Part, register_part
+from .base import Part, build_part, part_class, register_part
 
 
 def sum_partials(delta, dtype=None):
@@ -57,10 +58,36 @@ class StreamCopy:
         return None
 
 
+class StreamsPending:
+    """A sublayer's output `y` that the residual streams have not received yet (`resid` [tokens, streams * width], a token's
+    streams side by side): x_t <- sum_s mix[s, t] x_s + share[t] y, all streams at once. The next norm's kernel does that
+    on its way; `apply` does it alone."""
+
+    def __init__(self, y, mix, share):
+        self.y, self.mix, self.share = y, mix, share
+
+    def apply(self, resid):
+        kernels.hyper_norm(resid, self.share.numel(), self.y, self.mix, self.share)
+        return None
+
+
 def settle(resid, delta):
     """`delta` as something every norm takes: a pending :class:`PostNormed` is added to the stream now; a
     :class:`StreamCopy` has nothing to add."""
-    return delta.apply(resid) if isinstance(delta, (PostNormed, StreamCopy)) else delta
+    return delta.apply(resid) if isinstance(delta, (PostNormed, StreamCopy, StreamsPending)) else delta
+
+
+def read_streams(norm, resid, delta, n_streams: int, read=None, rows=None, write_back: bool = True):
+    """norm(sum_s read[s] x_s) of the residual streams `resid` (read None: the plain sum), after they have received `delta` (a
+    :class:`StreamsPending`, or None), in one launch. `rows` gathers source rows (the streams then stay as they are)."""
+    if delta is not None and not isinstance(delta, StreamsPending):
+        raise ConfigError("residual streams take the output of a block that has them")
+    y, mix, share = (delta.y, delta.mix, delta.share) if delta is not None else (None, None, None)
+    n = resid.shape[0] if rows is None else rows.numel()
+    out = torch.empty((n, norm.spec.size), dtype=norm.runtime.dtype, device=resid.device)
+    kernels.hyper_norm(resid, n_streams, y, mix, share, read, norm.gain, getattr(norm, "bias", None), norm.spec.eps,
+                       isinstance(norm, LayerNorm), out, rows=rows, write_back=write_back)
+    return out
 
 
 class RMSNorm(Part):
@@ -199,6 +226,39 @@ class LayerNorm(Part):
     __call__ = forward
 
 
+class GainLayerNorm(LayerNorm):
+    """Layer norm with a gain and no bias."""
+
+    @classmethod
+    def needs_of_spec(cls, spec):
+        return {spec.prefix: TensorNeed((spec.size,), "gain", "gain")}
+
+    def load(self, tensors):
+        self.gain = self._gain(tensors[self.spec.prefix])
+
+
+class StreamSumNorm(Part):
+    """The norm of the sum of a model's residual streams; what is pending joins them on the way."""
+
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        self.norm = build_part("norm", spec.norm, runtime)
+
+    @classmethod
+    def needs_of_spec(cls, spec):
+        return part_class("norm", spec.norm).needs_of_spec(spec.norm)
+
+    def load(self, tensors):
+        self.norm.load(tensors)
+
+    def forward(self, resid, delta, rows=None, write_resid=True):
+        return read_streams(self.norm, resid, delta, self.spec.streams, rows=rows, write_back=write_resid)
+
+    __call__ = forward
+
+
+register_part("norm", "layernorm_nobias", GainLayerNorm)
+register_part("norm", "stream_sum", StreamSumNorm)
 register_part("norm", "rmsnorm", RMSNorm)
 register_part("norm", "layernorm", LayerNorm)
 register_part("norm", "dyt", DynamicTanh)

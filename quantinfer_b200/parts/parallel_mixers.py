@@ -6,7 +6,7 @@ pages: its need is this mixer's `cache_need`. Everything else the branches keep 
 entry (when its `cache_need` is a StateNeed) and what a branch keeps beside its pages (`state_need`) are laid side by
 side in ONE row of 32-bit numbers, this mixer's `state_need`, and each branch is handed its part of it.
 
-With `out_norm_names` in the spec each branch's output first passes an RMS norm over the model width (a gain per branch),
+`branch_scales` weights the two outputs in their sum. With `out_norm_names` in the spec each branch's output first passes an RMS norm over the model width (a gain per branch),
 and `sum_scale` multiplies the sum; norms, factor and sum are one kernel, which also adds the partial sums of the
 branches' output projections.
 """
@@ -52,6 +52,8 @@ class ParallelMixers(Part):
             self._layout.append(spans)
         self._floats = at
         self.out_gains = None
+        if getattr(spec, "branch_scales", None) is not None and getattr(spec, "out_norm_names", None) is not None:
+            raise ConfigError("parallel_mixers: branch_scales come without norms on the outputs")
         names = getattr(spec, "out_norm_names", None)
         if names is not None and (len(names) != 2 or not getattr(spec, "hidden_size", None)):
             raise ConfigError("parallel_mixers: norms on the branches' outputs need two gain names and the model width")
@@ -101,7 +103,8 @@ class ParallelMixers(Part):
         if self.out_gains is not None:
             kernels.normed_sum(outs[0], outs[1], self.out_gains[0], self.out_gains[1], self.spec.out_norm_eps, scale, out)
         else:
-            kernels.scaled_sum(outs[0], outs[1], scale, scale, out)
+            left, right = getattr(self.spec, "branch_scales", None) or (1.0, 1.0)
+            kernels.scaled_sum(outs[0], outs[1], scale * left, scale * right, out)
         return out
 
 

@@ -17,6 +17,7 @@ between layers with the same angles.
 from __future__ import annotations
 
 import math
+from fractions import Fraction
 
 import torch
 
@@ -48,6 +49,24 @@ def direct_frequencies(spec):
     lo, hi = max(math.floor(where(fast)), 0), min(math.ceil(where(slow)), dims - 1)
     ramp = torch.clamp((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
     return (f / factor * ramp + f * (1.0 - ramp)).to(torch.float32), 0.1 * math.log(factor) + 1.0
+
+
+def distance_buckets(rows: int, reach) -> list:
+    """The table row of every distance 0, 1, ... up to the first that reads the last row (as every longer one does). Below
+    h = rows / 2 a distance has a row of its own; a distance n from there on reads row h + min(floor(ln(n / h) / ln(reach / h)
+    (rows - h)), rows - h - 1). It is at least m steps beyond row h when (n / h)^(rows - h) >= (reach / h)^m, which is
+    decided in whole numbers, so that no rounding of a logarithm moves a distance that falls on an edge."""
+    h, reach = rows // 2, Fraction(reach)
+    if rows < 2 or reach <= h:
+        raise ConfigError(f"a distance bias of {rows} rows needs at least two and a reach ({float(reach):g}) above half their number")
+    top, out = rows - h, list(range(h))
+    n, m = h, 0
+    while m < top - 1:
+        while m < top - 1 and Fraction(n, h) ** top >= (reach / h) ** (m + 1):
+            m += 1
+        out.append(h + m)
+        n += 1
+    return out if out and out[-1] == rows - 1 else out + [rows - 1]
 
 
 class RopeHalfSplit(Part):
