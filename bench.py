@@ -280,8 +280,39 @@ def lemotar_arithmetic(config, spec):
     return a
 
 
+def siditar_arithmetic(config, spec):
+    """The same for a model of the Siditar design: per layer run the projections of both branches (softmax attention: q, k, v,
+    out; gated linear attention: q, k, v, gate, the decay's low-rank pair of rank 16, out), the clamped feed-forward's three
+    matrices, attention over every earlier key, and the recurrence's multiply-adds (three a state element and token) with
+    the 32-bit state it reads and writes in a decode step. Layers of a loop count once a run."""
+    H, V = spec.hidden_size, spec.vocab_size
+    params = scan_flops = state_bytes = 0
+    rank, heads, order = 16, [], config.run_order()
+    for i in order:
+        layer = config.layers[i]
+        l, r = layer.left, layer.right
+        params += H * ((l.heads + l.kv_heads) * l.dim + l.kv_heads * l.vdim) + l.heads * l.vdim * H
+        params += H * (2 * r.heads * r.dim + 2 * r.heads * r.vdim + rank) + rank * r.heads * r.dim + r.heads * r.vdim * H
+        heads.append((l.heads, l.dim, l.vdim, l.kv_heads))
+        scan_flops += 6.0 * r.heads * r.dim * r.vdim
+        state_bytes += 2 * 4 * r.heads * r.dim * r.vdim
+        if layer.ff is not None:
+            params += 3 * H * layer.ff
+    a = dict(L=len(order), H=H, V=V, layer_params=params / len(order), stored_params=params)
+    a["weight_bytes"] = 2 * (params + V * H)
+    a["kv_bytes_per_token"] = 0
+    a["kv_bytes"] = lambda ctx: sum(2 * g * (d + dv) * ctx for _, d, dv, g in heads)
+    a["state_bytes"] = state_bytes
+    a["gemm_flops"] = lambda T, rows_=1: 2.0 * T * params + 2.0 * H * V * rows_
+    a["attn_flops"] = lambda T: sum(2.0 * h * (d + dv) * (T * (T + 1) / 2) for h, d, dv, _ in heads)
+    a["scan_flops"] = lambda T: scan_flops * T
+    return a
+
+
 def model_arithmetic(config, spec):
     """Parameter counts, bytes and flops of the configuration (every matrix bf16)."""
+    if type(config).__name__ == "SiditarConfig":
+        return siditar_arithmetic(config, spec)
     if type(config).__name__ == "LemotarConfig":
         return lemotar_arithmetic(config, spec)
     if type(config).__name__ == "KiruvikConfig":
@@ -678,6 +709,42 @@ def compare_lemotar(args):
     return compare_kiruvik(args, "Lemotar layers beside Dulotar layers of equal width", LEMOTAR_SIZES, lemotar_entries)
 
 
+# ---- the Siditar design beside Dulotar layers of equal width ------------------------------------------------------
+# (width, softmax heads / kv heads of 128, linear-attention heads of 64 x 128, clamped feed-forward of three matrices):
+# four layers of two branches over two residual streams; beside them the closest existing design, Dulotar (softmax
+# attention and linear attention with a constant decay side by side, layer norms before the sublayers), four layers of two
+# branches with the same heads, its chunk as long as the context, feed-forwards of two matrices that hold the same weights
+SIDITAR_SIZES = {
+    "2048": dict(width=2048, heads=16, kv=4, lheads=16, ff=5504, ff2=8256),
+    "4096": dict(width=4096, heads=32, kv=8, lheads=32, ff=8192, ff2=12288),
+    "5120": dict(width=5120, heads=40, kv=8, lheads=40, ff=13824, ff2=20736),
+}
+
+
+def siditar_entries(size):
+    z = SIDITAR_SIZES[size]
+    both = {"left": {"heads": z["heads"], "kv_heads": z["kv"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "bias_max": 512,
+                     "q_temp": {"coef": 0.1, "every": 1024}},
+            "right": {"heads": z["lheads"], "dim": 64, "vdim": 128, "tau": 16.0}, "left_scale": 1.0, "right_scale": 0.5}
+    new = dict(architecture="Siditar", vocab=COMPARE_VOCAB, width=z["width"], streams=2, norm={"eps": 1e-5},
+               layers=[{"type": "parallel", "mixer": both, "mlp": {"kind": "dense", "ff": z["ff"], "limit": 7.0}}] * COMPARE_LAYERS)
+    old_both = {"left": {"heads": z["heads"], "kv_heads": z["kv"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "conv": 4, "softcap": 50.0,
+                         "rot": {"base": 500000.0, "dims": 64}, "mask": {"size": 4096}},
+                "right": {"heads": z["lheads"], "dim": 64, "vdim": 128, "decay": [1.0 - 2.0 ** -(2 + 6 * i / z["lheads"]) for i in range(z["lheads"])]},
+                "left_scale": 1.0, "right_scale": 0.5}
+    old = dict(architecture="Dulotar", vocab=COMPARE_VOCAB, width=z["width"], norm={"eps": 1e-5}, embedding={"scale": 1.0}, canon={"taps": 4},
+               layers=[{"type": "parallel", "mixer": old_both, "mlp": {"kind": "dense", "ff": z["ff2"]}}] * COMPARE_LAYERS)
+    common = dict(seed=5, prompt_len=COMPARE_PROMPT, context=4096, batch=COMPARE_BATCH, points=())
+    return (dict(common, config=new, name=f"Siditar layers of width {size}"), dict(common, config=old, name=f"Dulotar layers of width {size}"))
+
+
+def compare_siditar(args):
+    """Prefill and decode throughput of four Siditar layers (softmax and gated linear attention side by side over two
+    residual streams, clamped feed-forwards) beside four Dulotar layers of the same width, and each kernel class of both
+    alone with its share of the roofline."""
+    return compare_kiruvik(args, "Siditar layers beside Dulotar layers of equal width", SIDITAR_SIZES, siditar_entries)
+
+
 def compare_kiruvik(args, title="Kiruvik layers beside dense GQA (Qwen3) layers of equal width", sizes=None, entries_of=None):
     """Prefill and decode throughput of four Kiruvik layers (attention and state-space mixers, dense and routed
     feed-forwards) beside four dense GQA layers of the same width, heads and vocabulary, and each kernel class of both
@@ -1013,7 +1080,7 @@ def main() -> int:
                     help="run one part only (for profiler captures of a small case)")
     ap.add_argument("--timeline", action="store_true",
                     help="build the kernels with their time stamps and print where a decode step's time goes, kernel by kernel")
-    ap.add_argument("--compare", nargs="?", const="bebuvik", default=None, choices=["bebuvik", "kiruvik", "dulotar", "lemotar"],
+    ap.add_argument("--compare", nargs="?", const="bebuvik", default=None, choices=["bebuvik", "kiruvik", "dulotar", "lemotar", "siditar"],
                     help="instead of the headline workload: layers of another design (default: the latent-attention design) "
                          "beside dense GQA layers of equal sizes")
     ap.add_argument("--compare-sizes", default=None, help="widths to compare, with commas between them (default: all)")
@@ -1042,7 +1109,7 @@ def main() -> int:
     torch.cuda.set_device(0)
     if args.compare:
         args.skip_points = args.skip_classes = True
-        run = {"kiruvik": compare_kiruvik, "dulotar": compare_dulotar, "bebuvik": compare_designs, "lemotar": compare_lemotar}[args.compare]
+        run = {"kiruvik": compare_kiruvik, "dulotar": compare_dulotar, "bebuvik": compare_designs, "lemotar": compare_lemotar, "siditar": compare_siditar}[args.compare]
         print(json.dumps(run(args)))
         return 0
     if args.only == "mixed":

@@ -1063,6 +1063,7 @@ extern "C" int qi_gemm_bf16_plan(int M, int N, int K, int allow_split, int* swap
         // enough CTAs to keep the weight stream busy on 148 SMs, at least 8 k blocks per split
         // (filling every resident slot with 6 or 9 splits was measured no faster than powers of two)
         while (allow_split && tiles * sp < 148 && sp * 2 <= 16 && kb_total / (sp * 2) >= 8) sp *= 2;
+        sp = (kb_total + (kb_total + sp - 1) / sp - 1) / ((kb_total + sp - 1) / sp);      // none without work (129 k blocks: 15 parts of 9)
     } else {
         const int sms = sm_count();
         double best = 1e30;
