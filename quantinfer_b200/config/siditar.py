@@ -196,7 +196,8 @@ class SiditarConfig:
                 q_temp=(l.temp_coef, l.temp_every) if l.temp_every is not None else None, distance_bias=l.bias_max)
             right = GatedLinearAttentionSpec(hidden_size=w, heads=r.heads, head_dim=r.dim, value_dim=r.vdim, tau=r.tau, norm_eps=eps,
                                              prefix=p + "mix.right.")
-            mixer = ParallelMixersSpec(left, right, prefix=p + "mix.", branch_scales=(layer.left_scale, layer.right_scale), hidden_size=w)
+            mixer = ParallelMixersSpec(left, right, prefix=p + "mix.", branch_scales=(layer.left_scale, layer.right_scale), hidden_size=w,
+                                       merged=True)
             ffn = ClampedGLUSpec(w, layer.ff, layer.limit, GLU_ALPHA, p + "mlp.") if layer.ff is not None else None
             layers.append(HyperLayerSpec(mixer_norm=norm(p + "norm1"), mixer=mixer, ffn_norm=norm(p + "norm2") if ffn is not None else None,
                                          ffn=ffn, streams=self.streams,

@@ -280,6 +280,8 @@ class ParallelMixersSpec:
     out_norm_eps: float = 1e-6
     sum_scale: float = 1.0
     hidden_size: Optional[int] = None  # needed with `out_norm_names` (the gains' size)
+    merged: bool = False               # the branches' first projections run as one product, and so do their output projections
+                                       # (over both branches' results side by side): for branches that offer `mix`
     branch_scales: Optional[tuple] = None  # (left, right): factors on the two outputs, without norms: left * a + right * b
 
 

@@ -39,7 +39,7 @@ attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const T* 
                          const int* __restrict__ positions, const int* __restrict__ token_req,
                          int nq, int nkv, int d, int dv, float scale, float softcap, float out_scale, int window, int chunk,
                          const T* __restrict__ gate, long long ldg, const float* __restrict__ sink, const float* __restrict__ bias, int bias_len,
-                         int* __restrict__ status) {
+                         long long ldo, int* __restrict__ status) {
     extern __shared__ float smem[];
     float* q_s = smem;                          // [d]
     float* part_acc = smem + d;                 // [kWarps][dv]
@@ -128,7 +128,7 @@ attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const T* 
         gl += part_l[w] * wscale[w];
     }
     if (sink) gl += expf(sink[h] - gm);
-    T* orow = out + ((size_t)t * nq + h) * dv;
+    T* orow = out + (size_t)t * ldo + (size_t)h * dv;
     const T* grow = gate ? gate + (size_t)t * ldg + (size_t)h * dv : nullptr;
     for (int i = threadIdx.x; i < dv; i += blockDim.x) {
         float o = 0.f;
@@ -147,13 +147,15 @@ attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const T* 
 // softcap c > 0: a score s becomes c tanh(s / c) before the softmax (0: scores as they are); out_scale multiplies the result.
 // sink (may be null): float32 [nq]; the softmax's denominator of head h holds exp(sink[h]) once more.
 // bias (may be null): float32 [nq, bias_len]; a key n positions back adds bias[h, min(n, bias_len - 1)] to its score.
+// ldo: elements from one row of out to the next.
 extern "C" int qi_attention_generic_bias(const void* q, void* out, int dtype, const void* k_pages,
                                        const void* v_pages, const int* block_table, int max_blocks,
                                        int page_size, int num_pages, const int* positions,
                                        const int* token_req, int n_tokens, int nq, int nkv, int d, int dv,
                                        float scale, float softcap, float out_scale, int window, int chunk, const void* gate,
-                                       long long ldg, const float* sink, const float* bias, int bias_len, int* status,
+                                       long long ldg, const float* sink, const float* bias, int bias_len, long long ldo, int* status,
                                        cudaStream_t stream) {
+    QI_REQUIRE(ldo >= (long long)nq * dv, "attention: the output's rows are too short");
     QI_REQUIRE(!bias || bias_len > 0, "attention: an empty distance bias");
     QI_REQUIRE(n_tokens >= 0 && nq > 0 && nkv > 0 && d > 0 && dv > 0, "attention: bad sizes");
     QI_REQUIRE(nq % nkv == 0, "attention: %d query heads are not a multiple of %d kv heads", nq, nkv);
@@ -171,10 +173,10 @@ extern "C" int qi_attention_generic_bias(const void* q, void* out, int dtype, co
         dim3 grid(nq, nt);
         QI_DISPATCH_DTYPE(dtype, T, {
             qi::launch(attention_generic_kernel<T>, grid, dim3(kWarps * 32), smem, stream,
-                (const T*)q + (size_t)t0 * nq * d, (T*)out + (size_t)t0 * nq * dv, (const T*)k_pages,
+                (const T*)q + (size_t)t0 * nq * d, (T*)out + (size_t)t0 * ldo, (const T*)k_pages,
                 (const T*)v_pages, block_table, max_blocks, page_size, num_pages, positions + t0,
                 token_req + t0, nq, nkv, d, dv, scale, softcap, out_scale, window, chunk,
-                gate ? (const T*)gate + (size_t)t0 * ldg : (const T*)nullptr, ldg, sink, bias, bias_len, status);
+                gate ? (const T*)gate + (size_t)t0 * ldg : (const T*)nullptr, ldg, sink, bias, bias_len, ldo, status);
         });
     }
     return qi::check_launch("attention_generic");
@@ -188,7 +190,7 @@ extern "C" int qi_attention_generic_sink(const void* q, void* out, int dtype, co
                                        long long ldg, const float* sink, int* status, cudaStream_t stream) {
     return qi_attention_generic_bias(q, out, dtype, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, positions,
                                      token_req, n_tokens, nq, nkv, d, dv, scale, softcap, out_scale, window, chunk, gate, ldg,
-                                     sink, nullptr, 0, status, stream);
+                                     sink, nullptr, 0, (long long)nq * dv, status, stream);
 }
 
 extern "C" int qi_attention_generic_cap(const void* q, void* out, int dtype, const void* k_pages,

@@ -264,7 +264,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                                       float scale_log2e, int window, int* __restrict__ status, int n_ranges,
                                       float* __restrict__ ws_o, float* __restrict__ ws_ml, int chunk,
                                       const qi::bf16* __restrict__ gate, long long ldg, float cap, float cap_pre,
-                                      float out_scale, const float* __restrict__ sink, const float* __restrict__ bias, int bias_len) {
+                                      float out_scale, const float* __restrict__ sink, const float* __restrict__ bias, int bias_len, long long ldo) {
     extern __shared__ uint8_t smem_raw[];
     using B = Bars;
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -573,7 +573,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
             // the sink: exp(sink_h) once more in the denominator (m is a base-2 exponent); with key ranges the merge adds it
             if (sink && m != -INFINITY) l += ex2(sink[h] * 1.4426950408889634f - m);
             const float inv = l > 0.f ? out_scale / l : 0.f;
-            qi::bf16* orow = out + ((size_t)(q0 + row) * nq + h) * D;
+            qi::bf16* orow = out + (size_t)(q0 + row) * ldo + (size_t)h * D;
             const qi::bf16* grow = gate ? gate + (size_t)(q0 + row) * ldg + (size_t)h * D : nullptr;
             // the row's 128 columns in two halves, each half's loads in flight together
 #pragma unroll 1
@@ -615,7 +615,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
 __global__ void attention_prefill_merge_kernel(const float* __restrict__ ws_o, const float* __restrict__ ws_ml,
                                                qi::bf16* __restrict__ out, int nq, int n_ranges,
                                                const qi::bf16* __restrict__ gate, long long ldg, float out_scale,
-                                               const float* __restrict__ sink) {
+                                               const float* __restrict__ sink, long long ldo) {
     qi::pdl_enter();
     const int h = blockIdx.x;
     const size_t t = blockIdx.y;
@@ -635,7 +635,7 @@ __global__ void attention_prefill_merge_kernel(const float* __restrict__ ws_o, c
         L += sink_term;
         float o = L > 0.f ? O / L * out_scale : 0.f;
         if (gate) o = o / (1.f + __expf(-__bfloat162float(gate[t * (size_t)ldg + (size_t)h * D + col])));
-        out[(t * nq + h) * D + col] = __float2bfloat16_rn(o);
+        out[t * (size_t)ldo + (size_t)h * D + col] = __float2bfloat16_rn(o);
     }
 }
 
@@ -689,14 +689,17 @@ extern "C" int qi_attention_prefill_tcgen05_supported(int nq, int nkv, int d, in
 // `ldg` elements apart; the output is multiplied element by element with its sigmoid. softcap c > 0: a score s (scale
 // applied) becomes c tanh(s / c) before the softmax. out_scale multiplies the result. sink (or null): float32 [nq]; the
 // softmax's denominator of head h holds exp(sink[h]) once more. bias (or null): float32 [nq, bias_len]; a key n positions
-// back adds bias[h, min(n, bias_len - 1)] to its score (after the cap).
+// back adds bias[h, min(n, bias_len - 1)] to its score (after the cap). ldo: elements from one row of out to the next.
 extern "C" int qi_attention_prefill_tcgen05_bias(const void* q, void* out, const void* k_pages, const void* v_pages,
                                                const int* block_table, int max_blocks, int page_size, int num_pages,
                                                const int* q_start, const int* start_pos, const int* tile_req,
                                                const int* tile_q0, int n_tiles, int n_tokens, int nq, int nkv, int d,
                                                float scale, int window, int chunk, const void* gate, long long ldg,
                                                int n_ranges, float* workspace, int* status, float softcap, float out_scale,
-                                               const float* sink, const float* bias, int bias_len, cudaStream_t stream) {
+                                               const float* sink, const float* bias, int bias_len, long long ldo,
+                                               cudaStream_t stream) {
+    QI_REQUIRE(ldo >= (long long)nq * D && ldo % 8 == 0 && ((uintptr_t)out & 15) == 0,
+               "attention_prefill_tcgen05: the output must be 16-byte aligned with rows a multiple of 8 elements apart");
     QI_REQUIRE(!bias || bias_len > 0, "attention_prefill_tcgen05: an empty distance bias");
     QI_REQUIRE(softcap >= 0.f && scale > 0.f, "attention_prefill_tcgen05: the soft cap must be >= 0 (0 = none) and the scale positive");
     QI_REQUIRE(chunk >= 0 && (!gate || (((uintptr_t)gate & 15) == 0 && ldg % 8 == 0 && ldg >= (long long)nq * D)),
@@ -731,11 +734,11 @@ extern "C" int qi_attention_prefill_tcgen05_bias(const void* q, void* out, const
     qi::launch(attention_prefill_tcgen05_kernel, dim3(nq, n_tiles, n_ranges), dim3(kThreads), kSmemBytes, stream, mq, mk, mv,
                (qi::bf16*)out, block_table, max_blocks, page_size, box_rows, num_pages, q_start, start_pos, tile_req,
                tile_q0, nq, nkv, softcap > 0.f ? log2e : scale * log2e, window, status, n_ranges, ws_o, ws_ml, chunk,
-               (const qi::bf16*)gate, ldg, softcap, cap_pre, out_scale, sink, bias, bias_len);
+               (const qi::bf16*)gate, ldg, softcap, cap_pre, out_scale, sink, bias, bias_len, ldo);
     if (n_ranges > 1) {
         if (int rc = qi::check_launch("attention_prefill_tcgen05")) return rc;
         qi::launch(attention_prefill_merge_kernel, dim3(nq, n_tokens), dim3(128), 0, stream, (const float*)ws_o,
-                   (const float*)ws_ml, (qi::bf16*)out, nq, n_ranges, (const qi::bf16*)gate, ldg, out_scale, sink);
+                   (const float*)ws_ml, (qi::bf16*)out, nq, n_ranges, (const qi::bf16*)gate, ldg, out_scale, sink, ldo);
         return qi::check_launch("attention_prefill_merge");
     }
     return qi::check_launch("attention_prefill_tcgen05");
@@ -750,7 +753,7 @@ extern "C" int qi_attention_prefill_tcgen05_ex(const void* q, void* out, const v
                                                cudaStream_t stream) {
     return qi_attention_prefill_tcgen05_bias(q, out, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, q_start,
                                              start_pos, tile_req, tile_q0, n_tiles, n_tokens, nq, nkv, d, scale, window, chunk,
-                                             gate, ldg, n_ranges, workspace, status, softcap, out_scale, nullptr, nullptr, 0, stream);
+                                             gate, ldg, n_ranges, workspace, status, softcap, out_scale, nullptr, nullptr, 0, (long long)nq * D, stream);
 }
 
 extern "C" int qi_attention_prefill_tcgen05(const void* q, void* out, const void* k_pages, const void* v_pages,

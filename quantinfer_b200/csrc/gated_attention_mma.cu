@@ -75,7 +75,7 @@ gated_attention_mma_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restrict_
                            int page_size, int num_pages, const int* __restrict__ q_start, const int* __restrict__ start_pos,
                            int n_entries, int nq, int nkv, int d, int dv, float scale_log2e, float softcap, float out_scale,
                            int window, int chunk, const qi::bf16* __restrict__ gate, long long ldg, const float* __restrict__ sink,
-                           const float* __restrict__ bias, int bias_len, int n_ranges, float* __restrict__ ws_o, float* __restrict__ ws_ml, int* __restrict__ status) {
+                           const float* __restrict__ bias, int bias_len, int n_ranges, float* __restrict__ ws_o, float* __restrict__ ws_ml, long long ldo, int* __restrict__ status) {
     extern __shared__ __align__(16) uint8_t smem_raw[];
     constexpr int SK = DK + kPad, SV = DV + kPad;
     qi::bf16* Qs = reinterpret_cast<qi::bf16*>(smem_raw);       // [kQT][SK]
@@ -305,8 +305,203 @@ gated_attention_mma_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restrict_
                 v0 = v0 / (1.0f + expf(-__bfloat162float(g[0])));
                 v1 = v1 / (1.0f + expf(-__bfloat162float(g[1])));
             }
-            *reinterpret_cast<__nv_bfloat162*>(out + (t * nq + h) * dv + col) = __floats2bfloat162_rn(v0 * out_scale, v1 * out_scale);
+            *reinterpret_cast<__nv_bfloat162*>(out + t * (size_t)ldo + (size_t)h * dv + col) = __floats2bfloat162_rn(v0 * out_scale, v1 * out_scale);
         }
+    }
+}
+
+// Steps of single tokens (every entry has one): the query heads that share a key head are the rows of one tile (up to 16
+// of them), so every key and value is read once a group and not once a query head. A CTA of four warps takes one entry, one
+// key head and one range of keys; each warp scores a quarter of every tile's 64 keys and keeps a reference, a sum and an
+// accumulator of its own, which meet in shared memory at the end (in warp order); with several ranges the merge
+// kernel adds the parts.
+constexpr int kGroupRows = 16;
+
+template <int DK, int DV>
+__global__ void __launch_bounds__(kThreads)
+gated_attention_decode_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restrict__ out, const qi::bf16* __restrict__ k_pages,
+                              const qi::bf16* __restrict__ v_pages, const int* __restrict__ block_table, int max_blocks,
+                              int page_size, int num_pages, const int* __restrict__ q_start, const int* __restrict__ start_pos,
+                              int nq, int nkv, int d, int dv, float scale_log2e, float softcap, float out_scale,
+                              int window, int chunk, const qi::bf16* __restrict__ gate, long long ldg, const float* __restrict__ sink,
+                              const float* __restrict__ bias, int bias_len, int n_ranges, float* __restrict__ ws_o,
+                              float* __restrict__ ws_ml, long long ldo, int* __restrict__ status) {
+    extern __shared__ __align__(16) uint8_t smem_raw[];
+    constexpr int SK = DK + kPad, SV = DV + kPad;
+    qi::bf16* Qs = reinterpret_cast<qi::bf16*>(smem_raw);       // [kGroupRows][SK]
+    qi::bf16* Kbuf = Qs + kGroupRows * SK;                       // 2 x [kKT][SK]
+    qi::bf16* Vbuf = Kbuf + 2 * kKT * SK;                        // 2 x [kKT][SV]
+    constexpr float kLog2e = 1.4426950408889634f;
+
+    qi::pdl_wait();
+    const int e = blockIdx.x, hk = blockIdx.y, group = nq / nkv, h0 = hk * group;
+    const int t = q_start[e], pos = start_pos[e];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int* table = block_table + (size_t)e * max_blocks;
+    int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    if (chunk > 0) lo = max(lo, pos / chunk * chunk);
+
+    bool bad_page = false;
+    auto request_tile = [&](int t0, int buf) {
+        auto page_row = [&](int r, const qi::bf16* pages, int width) -> const qi::bf16* {
+            const int key = t0 + r;
+            if (key < lo || key > pos) return nullptr;
+            const int page = table[key / page_size];
+            if (page < 0 || page >= num_pages) { bad_page = true; return nullptr; }
+            return pages + (((size_t)page * nkv + hk) * page_size + (key % page_size)) * (size_t)width;
+        };
+        fill_tile_async(Kbuf + (size_t)buf * kKT * SK, SK, kKT, d, DK, k_pages, [&](int r) { return page_row(r, k_pages, d); });
+        fill_tile_async(Vbuf + (size_t)buf * kKT * SV, SV, kKT, dv, DV, k_pages, [&](int r) { return page_row(r, v_pages, dv); });
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    int t_first = lo / kKT * kKT, t_last = pos;
+    if (n_ranges > 1) {
+        const int per = ((pos - t_first) / kKT + n_ranges) / n_ranges;
+        t_first += (int)blockIdx.z * per * kKT;
+        t_last = min(pos, t_first + per * kKT - 1);
+    }
+    int buf = 0;
+    if (t_first <= t_last) request_tile(t_first, 0);
+    fill_tile(Qs, SK, kGroupRows, d, DK, [&](int r) -> const qi::bf16* {
+        return r < group ? q + ((size_t)t * nq + h0 + r) * d : nullptr;
+    });
+    __syncthreads();
+    uint32_t qa[DK / 16][4];
+    const int rA = lane >> 2, rB = rA + 8;
+    {
+        const int c = (lane & 3) * 2;
+#pragma unroll
+        for (int kk = 0; kk < DK / 16; ++kk) {
+            qa[kk][0] = *reinterpret_cast<const uint32_t*>(Qs + (size_t)rA * SK + kk * 16 + c);
+            qa[kk][1] = *reinterpret_cast<const uint32_t*>(Qs + (size_t)rB * SK + kk * 16 + c);
+            qa[kk][2] = *reinterpret_cast<const uint32_t*>(Qs + (size_t)rA * SK + kk * 16 + 8 + c);
+            qa[kk][3] = *reinterpret_cast<const uint32_t*>(Qs + (size_t)rB * SK + kk * 16 + 8 + c);
+        }
+    }
+    const bool inA = rA < group, inB = rB < group;
+    const float* biasA = bias ? bias + (size_t)(h0 + (inA ? rA : 0)) * bias_len : nullptr;
+    const float* biasB = bias ? bias + (size_t)(h0 + (inB ? rB : 0)) * bias_len : nullptr;
+    float mA = -INFINITY, mB = -INFINITY, lA = 0.f, lB = 0.f;
+    float o[DV / 8][4];
+#pragma unroll
+    for (int n = 0; n < DV / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+
+    for (int t0 = t_first; t0 <= t_last; t0 += kKT, buf ^= 1) {
+        if (t0 + kKT <= t_last) {        // the next tile lands while this one is multiplied
+            request_tile(t0 + kKT, buf ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        const qi::bf16* Ks = Kbuf + (size_t)buf * kKT * SK + (size_t)warp * 16 * SK;
+        const qi::bf16* Vs = Vbuf + (size_t)buf * kKT * SV + (size_t)warp * 16 * SV;
+        const int k0 = t0 + warp * 16;
+        float s[2][4];
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+            s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+            const qi::bf16* kr = Ks + (size_t)(n * 8 + (lane >> 2)) * SK + (lane & 3) * 2;
+#pragma unroll
+            for (int kk = 0; kk < DK / 16; ++kk)
+                mma_bf16(s[n], qa[kk], *reinterpret_cast<const uint32_t*>(kr + kk * 16), *reinterpret_cast<const uint32_t*>(kr + kk * 16 + 8));
+        }
+        float tmA = -INFINITY, tmB = -INFINITY;
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                const int key = k0 + n * 8 + (lane & 3) * 2 + j;
+                float a = s[n][j] * scale_log2e, b = s[n][2 + j] * scale_log2e;
+                if (softcap > 0.f) {
+                    const float c = softcap * kLog2e;
+                    a = c * tanhf(a / c);
+                    b = c * tanhf(b / c);
+                }
+                const bool visible = key >= lo && key <= pos;
+                if (bias) {
+                    const int back = min(max(pos - key, 0), bias_len - 1);
+                    a = fmaf(__ldg(biasA + back), kLog2e, a);
+                    b = fmaf(__ldg(biasB + back), kLog2e, b);
+                }
+                s[n][j] = visible && inA ? a : -INFINITY;
+                s[n][2 + j] = visible && inB ? b : -INFINITY;
+                tmA = fmaxf(tmA, s[n][j]);
+                tmB = fmaxf(tmB, s[n][2 + j]);
+            }
+        }
+        tmA = fmaxf(tmA, __shfl_xor_sync(0xffffffffu, tmA, 1)); tmA = fmaxf(tmA, __shfl_xor_sync(0xffffffffu, tmA, 2));
+        tmB = fmaxf(tmB, __shfl_xor_sync(0xffffffffu, tmB, 1)); tmB = fmaxf(tmB, __shfl_xor_sync(0xffffffffu, tmB, 2));
+        const float nmA = fmaxf(mA, tmA), nmB = fmaxf(mB, tmB);
+        const float baseA = nmA == -INFINITY ? 0.f : nmA, baseB = nmB == -INFINITY ? 0.f : nmB;
+        const float cA = exp2f(mA - baseA), cB = exp2f(mB - baseB);       // m = -inf gives 0
+        mA = nmA; mB = nmB;
+        float sumA = 0.f, sumB = 0.f;
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+            s[n][0] = exp2f(s[n][0] - baseA); s[n][1] = exp2f(s[n][1] - baseA);
+            s[n][2] = exp2f(s[n][2] - baseB); s[n][3] = exp2f(s[n][3] - baseB);
+            sumA += s[n][0] + s[n][1];
+            sumB += s[n][2] + s[n][3];
+        }
+        lA = lA * cA + sumA;      // the four lanes of a row keep partial sums; they meet at the end
+        lB = lB * cB + sumB;
+#pragma unroll
+        for (int n = 0; n < DV / 8; ++n) { o[n][0] *= cA; o[n][1] *= cA; o[n][2] *= cB; o[n][3] *= cB; }
+        const uint32_t pa[4] = {pack_bf16(s[0][0], s[0][1]), pack_bf16(s[0][2], s[0][3]), pack_bf16(s[1][0], s[1][1]), pack_bf16(s[1][2], s[1][3])};
+#pragma unroll
+        for (int n2 = 0; n2 < DV / 16; ++n2) {
+            uint32_t b0, b1, b2, b3;
+            const qi::bf16* vr = Vs + (size_t)(lane & 15) * SV + n2 * 16 + (lane >> 4) * 8;
+            const uint32_t addr = (uint32_t)__cvta_generic_to_shared(vr);
+            asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+                         : "=r"(b0), "=r"(b1), "=r"(b2), "=r"(b3) : "r"(addr));
+            mma_bf16(o[2 * n2], pa, b0, b1);
+            mma_bf16(o[2 * n2 + 1], pa, b2, b3);
+        }
+        __syncthreads();                 // every warp is done with this buffer before the tile after next is requested into it
+    }
+    if (bad_page && status) atomicOr(status, qi::kStatusBadPage);
+    lA += __shfl_xor_sync(0xffffffffu, lA, 1); lA += __shfl_xor_sync(0xffffffffu, lA, 2);
+    lB += __shfl_xor_sync(0xffffffffu, lB, 1); lB += __shfl_xor_sync(0xffffffffu, lB, 2);
+    // the warps' parts meet in shared memory (the tiles' space: 4 x 16 rows of DV + 2 numbers fit there for every DK)
+    static_assert(2 * kKT * (SK + SV) * 2 >= 4 * kGroupRows * (DV + 2) * 4, "the parts must fit the tiles' space");
+    float* So = reinterpret_cast<float*>(Kbuf);                   // [4][kGroupRows][DV]
+    float* Sm = So + 4 * kGroupRows * DV;                         // [4][kGroupRows][2]
+    if ((lane & 3) == 0) {
+        Sm[(warp * kGroupRows + rA) * 2] = mA; Sm[(warp * kGroupRows + rA) * 2 + 1] = lA;
+        Sm[(warp * kGroupRows + rB) * 2] = mB; Sm[(warp * kGroupRows + rB) * 2 + 1] = lB;
+    }
+#pragma unroll
+    for (int n = 0; n < DV / 8; ++n) {
+        const int col = n * 8 + (lane & 3) * 2;
+        *reinterpret_cast<float2*>(So + (size_t)(warp * kGroupRows + rA) * DV + col) = make_float2(o[n][0], o[n][1]);
+        *reinterpret_cast<float2*>(So + (size_t)(warp * kGroupRows + rB) * DV + col) = make_float2(o[n][2], o[n][3]);
+    }
+    __syncthreads();
+    for (int idx = threadIdx.x; idx < group * dv; idx += kThreads) {
+        const int r = idx / dv, col = idx % dv, h = h0 + r;
+        float M = -INFINITY;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) M = fmaxf(M, Sm[(w * kGroupRows + r) * 2]);
+        float L = 0.f, O = 0.f;
+#pragma unroll
+        for (int w = 0; w < 4; ++w) {
+            const float mw = Sm[(w * kGroupRows + r) * 2];
+            const float f = mw == -INFINITY ? 0.f : exp2f(mw - M);
+            L = fmaf(Sm[(w * kGroupRows + r) * 2 + 1], f, L);
+            O = fmaf(So[(size_t)(w * kGroupRows + r) * DV + col], f, O);
+        }
+        if (n_ranges > 1) {
+            const size_t slot = ((size_t)t * nq + h) * n_ranges + blockIdx.z;
+            if (col == 0) { ws_ml[slot * 2] = M; ws_ml[slot * 2 + 1] = L; }
+            ws_o[slot * dv + col] = O;
+            continue;
+        }
+        if (sink && M != -INFINITY) L += exp2f(sink[h] * kLog2e - M);
+        float v = L > 0.f ? O / L : 0.f;
+        if (gate) v = v / (1.0f + expf(-__bfloat162float(gate[(size_t)t * ldg + (size_t)h * dv + col])));
+        out[(size_t)t * ldo + (size_t)h * dv + col] = __float2bfloat16_rn(v * out_scale);
     }
 }
 
@@ -314,7 +509,7 @@ gated_attention_mma_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restrict_
 // the parts of a row that the key ranges left, added in range order.
 __global__ void gated_attention_merge_kernel(const float* __restrict__ ws_o, const float* __restrict__ ws_ml, qi::bf16* __restrict__ out,
                                              int nq, int dv, int n_ranges, const qi::bf16* __restrict__ gate, long long ldg,
-                                             const float* __restrict__ sink, float out_scale) {
+                                             const float* __restrict__ sink, float out_scale, long long ldo) {
     qi::pdl_wait();
     const int h = blockIdx.x;
     const size_t t = blockIdx.y;
@@ -333,7 +528,7 @@ __global__ void gated_attention_merge_kernel(const float* __restrict__ ws_o, con
         }
         float v = L > 0.f ? O / L : 0.f;
         if (gate) v = v / (1.0f + expf(-__bfloat162float(gate[t * (size_t)ldg + (size_t)h * dv + col])));
-        out[(t * nq + h) * dv + col] = __float2bfloat16_rn(v * out_scale);
+        out[t * (size_t)ldo + (size_t)h * dv + col] = __float2bfloat16_rn(v * out_scale);
     }
 }
 
@@ -343,20 +538,28 @@ template <int DK, int DV>
 int launch_one(dim3 grid, cudaStream_t stream, const void* q, void* out, const void* k_pages, const void* v_pages,
                const int* block_table, int max_blocks, int page_size, int num_pages, const int* q_start, const int* start_pos,
                int n_entries, int nq, int nkv, int d, int dv, float scale_log2e, float softcap, float out_scale, int window, int chunk,
-               const void* gate, long long ldg, const float* sink, const float* bias, int bias_len, int n_ranges, float* ws_o, float* ws_ml, int n_tokens, int* status) {
-    const size_t smem = sizeof(qi::bf16) * ((size_t)(kQT + 2 * kKT) * (DK + kPad) + (size_t)2 * kKT * (DV + kPad));
-    static bool raised = false;
-    if (!raised && smem > 48 * 1024) {
-        cudaFuncSetAttribute(gated_attention_mma_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        raised = true;
+               const void* gate, long long ldg, const float* sink, const float* bias, int bias_len, int n_ranges, float* ws_o, float* ws_ml, int n_tokens, int grouped, long long ldo, int* status) {
+    const size_t smem = sizeof(qi::bf16) * ((size_t)((grouped ? kGroupRows : kQT) + 2 * kKT) * (DK + kPad) + (size_t)2 * kKT * (DV + kPad));
+    static bool raised[2] = {false, false};
+    if (!raised[grouped] && smem > 48 * 1024) {
+        if (grouped) cudaFuncSetAttribute(gated_attention_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        else cudaFuncSetAttribute(gated_attention_mma_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        raised[grouped] = true;
     }
-    qi::launch(gated_attention_mma_kernel<DK, DV>, grid, dim3(kThreads), smem, stream, (const qi::bf16*)q, (qi::bf16*)out,
-               (const qi::bf16*)k_pages, (const qi::bf16*)v_pages, block_table, max_blocks, page_size, num_pages, q_start, start_pos,
-               n_entries, nq, nkv, d, dv, scale_log2e, softcap, out_scale, window, chunk, (const qi::bf16*)gate, ldg, sink, bias, bias_len, n_ranges, ws_o, ws_ml, status);
+    if (grouped)
+        qi::launch(gated_attention_decode_kernel<DK, DV>, grid, dim3(kThreads), smem, stream, (const qi::bf16*)q, (qi::bf16*)out,
+                   (const qi::bf16*)k_pages, (const qi::bf16*)v_pages, block_table, max_blocks, page_size, num_pages, q_start, start_pos,
+                   nq, nkv, d, dv, scale_log2e, softcap, out_scale, window, chunk, (const qi::bf16*)gate, ldg, sink, bias, bias_len, n_ranges,
+                   ws_o, ws_ml, ldo, status);
+    else
+        qi::launch(gated_attention_mma_kernel<DK, DV>, grid, dim3(kThreads), smem, stream, (const qi::bf16*)q, (qi::bf16*)out,
+                   (const qi::bf16*)k_pages, (const qi::bf16*)v_pages, block_table, max_blocks, page_size, num_pages, q_start, start_pos,
+                   n_entries, nq, nkv, d, dv, scale_log2e, softcap, out_scale, window, chunk, (const qi::bf16*)gate, ldg, sink, bias, bias_len,
+                   n_ranges, ws_o, ws_ml, ldo, status);
     if (n_ranges > 1) {
         if (int rc = qi::check_launch("gated_attention_mma")) return rc;
         qi::launch(gated_attention_merge_kernel, dim3(nq, n_tokens), dim3(128), 0, stream, (const float*)ws_o, (const float*)ws_ml,
-                   (qi::bf16*)out, nq, dv, n_ranges, (const qi::bf16*)gate, ldg, sink, out_scale);
+                   (qi::bf16*)out, nq, dv, n_ranges, (const qi::bf16*)gate, ldg, sink, out_scale, ldo);
         return qi::check_launch("gated_attention_merge");
     }
     return qi::check_launch("gated_attention_mma");
@@ -373,14 +576,19 @@ extern "C" int qi_gated_attention_mma_supported(int nq, int nkv, int d, int dv) 
 // softcap c > 0: a score s becomes c tanh(s / c) before the softmax; out_scale multiplies the result. sink (may be null):
 // float32 [nq]; the softmax's denominator of head h holds exp(sink[h]) once more.
 // bias (may be null): float32 [nq, bias_len]; a key n positions back adds bias[h, min(n, bias_len - 1)] to its score.
+// grouped: every entry has one token, and the query heads of a key head (up to 16) are the rows of one tile. ldo: elements from
+// one row of out to the next (even).
 // n_ranges > 1 (steps of single tokens over long contexts): every query tile's keys are cut into that many ranges over
 // separate CTAs and a second kernel adds the parts; `workspace` must then hold n_tokens * nq * n_ranges * (dv + 2) floats.
 extern "C" int qi_gated_attention_mma_bias(const void* q, void* out, const void* k_pages, const void* v_pages, const int* block_table,
                                       int max_blocks, int page_size, int num_pages, const int* q_start, const int* start_pos,
                                       int n_entries, int n_tokens, int nq, int nkv, int d, int dv, float scale, float softcap,
                                       float out_scale, int window, int chunk, const void* gate, long long ldg, const float* sink,
-                                      const float* bias, int bias_len, int n_ranges, float* workspace, int* status,
-                                      cudaStream_t stream) {
+                                      const float* bias, int bias_len, int n_ranges, float* workspace, int grouped, long long ldo,
+                                      int* status, cudaStream_t stream) {
+    QI_REQUIRE(ldo >= (long long)nq * dv && ldo % 2 == 0 && ((uintptr_t)out & 3) == 0, "gated_attention_mma: the output's rows are too short or odd");
+    QI_REQUIRE(!grouped || (n_tokens == n_entries && nkv > 0 && nq / nkv <= kGroupRows && nkv <= 65535),
+               "gated_attention_mma: the grouped form takes steps of single tokens and up to %d query heads a key head", kGroupRows);
     QI_REQUIRE(!bias || bias_len > 0, "gated_attention_mma: an empty distance bias");
     QI_REQUIRE(n_ranges >= 1 && n_ranges <= 64 && (n_ranges == 1 || (workspace && n_tokens <= 65535)), "gated_attention_mma: key ranges need a workspace (1 to 64 ranges, at most 65535 tokens)");
     QI_REQUIRE(qi_gated_attention_mma_supported(nq, nkv, d, dv), "gated_attention_mma: heads %d/%d of %d/%d are not covered", nq, nkv, d, dv);
@@ -390,13 +598,14 @@ extern "C" int qi_gated_attention_mma_bias(const void* q, void* out, const void*
     QI_REQUIRE(!gate || (ldg >= (long long)nq * dv && ldg % 2 == 0), "gated_attention_mma: the gate's rows are too short or odd");
     QI_REQUIRE(nq <= 65535, "gated_attention_mma: too many heads");
     if (n_tokens == 0 || n_entries == 0) return 0;
-    const dim3 grid(n_tokens / kQT + n_entries, nq, n_ranges);
+    grouped = grouped ? 1 : 0;
+    const dim3 grid(grouped ? n_entries : n_tokens / kQT + n_entries, grouped ? nkv : nq, n_ranges);
     float* ws_o = workspace;
     float* ws_ml = workspace ? workspace + (size_t)n_tokens * nq * n_ranges * dv : nullptr;
     const float sl = scale * 1.4426950408889634f;
 #define QI_GA(DKP, DVP)                                                                                                      \
     return launch_one<DKP, DVP>(grid, stream, q, out, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, q_start, \
-                                start_pos, n_entries, nq, nkv, d, dv, sl, softcap, out_scale, window, chunk, gate, ldg, sink, bias, bias_len, n_ranges, ws_o, ws_ml, n_tokens, status)
+                                start_pos, n_entries, nq, nkv, d, dv, sl, softcap, out_scale, window, chunk, gate, ldg, sink, bias, bias_len, n_ranges, ws_o, ws_ml, n_tokens, grouped, ldo, status)
 #define QI_GA_ROW(DKP)                                   \
     switch (padded(dv)) {                                \
         case 32: QI_GA(DKP, 32);                         \
@@ -437,5 +646,5 @@ extern "C" int qi_gated_attention_mma_sink(const void* q, void* out, const void*
                                       int* status, cudaStream_t stream) {
     return qi_gated_attention_mma_bias(q, out, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, q_start, start_pos,
                                          n_entries, n_tokens, nq, nkv, d, dv, scale, softcap, out_scale, window, chunk, gate, ldg, sink, nullptr, 0, 1,
-                                         nullptr, status, stream);
+                                         nullptr, 0, (long long)nq * dv, status, stream);
 }

@@ -205,7 +205,18 @@ struct RopeEpilogue {
     float eps;
     int max_blocks, page_size, num_pages, nq, nkv;
     int table_positions;     // rows of cos_t / sin_t
+    float limit, alpha;      // EPI = 3 (nothing else of this struct is used there)
 };
+
+// The activation of a (gate, up) pair: EPI 1 silu(g) u; EPI 3 the clamped form g sigmoid(alpha g) (u + 1) with g = min(gate,
+// limit), u = clamp(up, -limit, limit).
+template <int EPI>
+__device__ __forceinline__ float pair_act(float g, float u, const RopeEpilogue& e) {
+    if (EPI == 1) return silu_mul(g, u);
+    g = fminf(g, e.limit);
+    u = fminf(fmaxf(u, -e.limit), e.limit);
+    return g / (1.0f + expf(-e.alpha * g)) * (u + 1.0f);
+}
 
 __device__ __forceinline__ uint32_t pack2(float a, float b) {
     __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
@@ -325,6 +336,7 @@ __device__ __forceinline__ void rope_epilogue(uint32_t tmem_tile, int col_base, 
 
 // EPI = 0: store the product. EPI = 1: the product's columns come in pairs (gate, up) and
 // the kernel stores silu(gate) * up, half as wide (the feed-forward's activation fused in).
+// EPI = 3: the same pairs through the clamped gated form.
 // EPI = 2 (operands not swapped): the product is the q/k/v projection and `rope` says where
 // its heads go (q/k norm, rotation and the cache write fused in; `out` is not used).
 //
@@ -541,14 +553,14 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                     if (lane == 0) mbar_arrive(acc_empty_bar(acc));
                 }
                 const int b0 = tile_b * BN + c0;
-                if (SWAP && EPI == 1) {
+                if (SWAP && (EPI == 1 || EPI == 3)) {
                     // rows of A come in pairs (gate, up): even lanes hold gate, their neighbours up
 #pragma unroll
                     for (int q = 0; q < kChunk; ++q) {
                         const float mine = __uint_as_float(r[q]);
                         const float other = __shfl_xor_sync(0xffffffffu, mine, 1);
                         if ((lane & 1) == 0 && a_row + 1 < rows_a && b0 + q < rows_b)
-                            store1<TOut>(obase + (size_t)(b0 + q) * ld_out + (a_row >> 1), silu_mul(mine, other));
+                            store1<TOut>(obase + (size_t)(b0 + q) * ld_out + (a_row >> 1), pair_act<EPI>(mine, other, rope));
                     }
                 } else if (SWAP) {
                     // out[b, a]: for a fixed column the warp's lanes write consecutive addresses
@@ -557,7 +569,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                         for (int q = 0; q < kChunk; ++q)
                             if (b0 + q < rows_b) store1<TOut>(obase + (size_t)(b0 + q) * ld_out + a_row, __uint_as_float(r[q]));
                     }
-                } else if (EPI == 1) {
+                } else if (EPI == 1 || EPI == 3) {
                     if (a_row < rows_a) {
                         TOut* orow = obase + (size_t)a_row * ld_out + (b0 >> 1);
                         const bool full = b0 + kChunk <= rows_b;
@@ -570,8 +582,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 #pragma unroll
                                 for (int q = 0; q < 4; ++q) {
                                     __nv_bfloat162 pr = __floats2bfloat162_rn(
-                                        silu_mul(__uint_as_float(r[q0 + 4 * q]), __uint_as_float(r[q0 + 4 * q + 1])),
-                                        silu_mul(__uint_as_float(r[q0 + 4 * q + 2]), __uint_as_float(r[q0 + 4 * q + 3])));
+                                        pair_act<EPI>(__uint_as_float(r[q0 + 4 * q]), __uint_as_float(r[q0 + 4 * q + 1]), rope),
+                                        pair_act<EPI>(__uint_as_float(r[q0 + 4 * q + 2]), __uint_as_float(r[q0 + 4 * q + 3]), rope));
                                     vw[q] = *reinterpret_cast<uint32_t*>(&pr);
                                 }
                                 *reinterpret_cast<uint4*>(reinterpret_cast<qi::bf16*>(orow) + (q0 >> 1)) = v;
@@ -580,7 +592,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 #pragma unroll
                             for (int q = 0; q < kChunk; q += 2)
                                 if (b0 + q + 1 < rows_b)
-                                    store1<TOut>(orow + (q >> 1), silu_mul(__uint_as_float(r[q]), __uint_as_float(r[q + 1])));
+                                    store1<TOut>(orow + (q >> 1), pair_act<EPI>(__uint_as_float(r[q]), __uint_as_float(r[q + 1]), rope));
                         }
                     }
                 } else {
@@ -871,28 +883,28 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid
                 const int b0 = tile_n * TN + c0;
                 if (row >= rows_a) continue;
                 const bool full = b0 + 32 <= rows_b;
-                if (EPI == 1) {
+                if (EPI == 1 || EPI == 3) {
                     // columns come in pairs (gate, up): half as many outputs
                     TOut* orow = obase + (size_t)row * ld_out + (b0 >> 1);
                     if (full && ((reinterpret_cast<uintptr_t>(orow) & 15u) == 0) && sizeof(TOut) == 2) {
 #pragma unroll
                         for (int q0 = 0; q0 < 32; q0 += 16) {
                             uint4 v;
-                            v.x = pack2(silu_mul(__uint_as_float(r[q0 + 0]), __uint_as_float(r[q0 + 1])),
-                                        silu_mul(__uint_as_float(r[q0 + 2]), __uint_as_float(r[q0 + 3])));
-                            v.y = pack2(silu_mul(__uint_as_float(r[q0 + 4]), __uint_as_float(r[q0 + 5])),
-                                        silu_mul(__uint_as_float(r[q0 + 6]), __uint_as_float(r[q0 + 7])));
-                            v.z = pack2(silu_mul(__uint_as_float(r[q0 + 8]), __uint_as_float(r[q0 + 9])),
-                                        silu_mul(__uint_as_float(r[q0 + 10]), __uint_as_float(r[q0 + 11])));
-                            v.w = pack2(silu_mul(__uint_as_float(r[q0 + 12]), __uint_as_float(r[q0 + 13])),
-                                        silu_mul(__uint_as_float(r[q0 + 14]), __uint_as_float(r[q0 + 15])));
+                            v.x = pack2(pair_act<EPI>(__uint_as_float(r[q0 + 0]), __uint_as_float(r[q0 + 1]), rope),
+                                        pair_act<EPI>(__uint_as_float(r[q0 + 2]), __uint_as_float(r[q0 + 3]), rope));
+                            v.y = pack2(pair_act<EPI>(__uint_as_float(r[q0 + 4]), __uint_as_float(r[q0 + 5]), rope),
+                                        pair_act<EPI>(__uint_as_float(r[q0 + 6]), __uint_as_float(r[q0 + 7]), rope));
+                            v.z = pack2(pair_act<EPI>(__uint_as_float(r[q0 + 8]), __uint_as_float(r[q0 + 9]), rope),
+                                        pair_act<EPI>(__uint_as_float(r[q0 + 10]), __uint_as_float(r[q0 + 11]), rope));
+                            v.w = pack2(pair_act<EPI>(__uint_as_float(r[q0 + 12]), __uint_as_float(r[q0 + 13]), rope),
+                                        pair_act<EPI>(__uint_as_float(r[q0 + 14]), __uint_as_float(r[q0 + 15]), rope));
                             *reinterpret_cast<uint4*>(reinterpret_cast<qi::bf16*>(orow) + (q0 >> 1)) = v;
                         }
                     } else {
 #pragma unroll
                         for (int q = 0; q < 32; q += 2)
                             if (b0 + q + 1 < rows_b)
-                                store1<TOut>(orow + (q >> 1), silu_mul(__uint_as_float(r[q]), __uint_as_float(r[q + 1])));
+                                store1<TOut>(orow + (q >> 1), pair_act<EPI>(__uint_as_float(r[q]), __uint_as_float(r[q + 1]), rope));
                     }
                 } else {
                     TOut* orow = obase + (size_t)row * ld_out + b0;
@@ -953,11 +965,12 @@ EncodeTiledFn get_encode() {
 }
 
 // Map of a row-major bf16 matrix [rows, K] with boxes of [box_rows, 64] and the 128-byte swizzle.
-int make_map(CUtensorMap* map, const void* ptr, int rows, int K, int box_rows) {
+// rows of K numbers, `ld` apart (0: K)
+int make_map(CUtensorMap* map, const void* ptr, int rows, int K, int box_rows, long long ld = 0) {
     EncodeTiledFn enc = get_encode();
     if (!enc) return qi::fail("gemm_bf16: cuTensorMapEncodeTiled is not available from the driver");
     cuuint64_t dims[2] = {(cuuint64_t)K, (cuuint64_t)rows};
-    cuuint64_t strides[1] = {(cuuint64_t)K * 2};
+    cuuint64_t strides[1] = {(cuuint64_t)(ld ? ld : K) * 2};
     cuuint32_t box[2] = {(cuuint32_t)BK, (cuuint32_t)box_rows};
     cuuint32_t estr[2] = {1, 1};
     CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims, strides, box, estr,
@@ -1026,13 +1039,14 @@ constexpr int stages_of(int bn) { return bn <= 16 ? 6 : bn == 32 ? 5 : bn == 128
 
 template <bool SWAP, typename TOut, int EPI = 0>
 int launch_bn(int bn, const CUtensorMap& ma, const CUtensorMap& mb, TOut* out, int rows_a, int rows_b, int K,
-              long long ld, int splits, int kb_per_split, long long split_stride, int* status, cudaStream_t stream) {
+              long long ld, int splits, int kb_per_split, long long split_stride, int* status, cudaStream_t stream,
+              const RopeEpilogue& rope = RopeEpilogue{}) {
     switch (bn) {
-        case 16: return launch<16, stages_of(16), SWAP, TOut, EPI>(ma, mb, out, rows_a, rows_b, K, ld, splits, kb_per_split, split_stride, status, stream);
-        case 32: return launch<32, stages_of(32), SWAP, TOut, EPI>(ma, mb, out, rows_a, rows_b, K, ld, splits, kb_per_split, split_stride, status, stream);
-        case 64: return launch<64, stages_of(64), SWAP, TOut, EPI>(ma, mb, out, rows_a, rows_b, K, ld, splits, kb_per_split, split_stride, status, stream);
-        case 128: return launch<128, stages_of(128), SWAP, TOut, EPI>(ma, mb, out, rows_a, rows_b, K, ld, splits, kb_per_split, split_stride, status, stream);
-        case 256: return launch<256, stages_of(256), SWAP, TOut, EPI>(ma, mb, out, rows_a, rows_b, K, ld, splits, kb_per_split, split_stride, status, stream);
+        case 16: return launch<16, stages_of(16), SWAP, TOut, EPI>(ma, mb, out, rows_a, rows_b, K, ld, splits, kb_per_split, split_stride, status, stream, rope);
+        case 32: return launch<32, stages_of(32), SWAP, TOut, EPI>(ma, mb, out, rows_a, rows_b, K, ld, splits, kb_per_split, split_stride, status, stream, rope);
+        case 64: return launch<64, stages_of(64), SWAP, TOut, EPI>(ma, mb, out, rows_a, rows_b, K, ld, splits, kb_per_split, split_stride, status, stream, rope);
+        case 128: return launch<128, stages_of(128), SWAP, TOut, EPI>(ma, mb, out, rows_a, rows_b, K, ld, splits, kb_per_split, split_stride, status, stream, rope);
+        case 256: return launch<256, stages_of(256), SWAP, TOut, EPI>(ma, mb, out, rows_a, rows_b, K, ld, splits, kb_per_split, split_stride, status, stream, rope);
     }
     return qi::fail("gemm_bf16: no kernel for a tile width of %d", bn);
 }
@@ -1116,23 +1130,28 @@ extern "C" int qi_gemm_bf16_plan(int M, int N, int K, int allow_split, int* swap
 // With splits > 1, `workspace` must hold splits * M * N floats.
 // epilogue 1: w's rows come in (gate, up) pairs and out[M, N / 2] = silu(gate) * up (bf16, no split).
 // out may be null with splits > 1: the partial sums stay in the workspace for the consumer.
-extern "C" int qi_gemm_bf16(const void* x, const void* w, void* out, int out_dtype, int M, int N, int K,
-                            int swap, int bn, int splits, int epilogue, void* workspace, int* status,
-                            cudaStream_t stream) {
+// epilogue 3: the same pairs through g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit).
+// ldx: elements from one row of x to the next (a block of columns of wider rows; 0: K).
+extern "C" int qi_gemm_bf16_ex(const void* x, long long ldx, const void* w, void* out, int out_dtype, int M, int N, int K,
+                               int swap, int bn, int splits, int epilogue, float limit, float alpha, void* workspace,
+                               int* status, cudaStream_t stream) {
+    QI_REQUIRE(ldx == 0 || (ldx >= K && ldx % 8 == 0), "gemm_bf16: rows of x must lie a multiple of 8 elements apart, at least K");
     QI_REQUIRE(M > 0 && N > 0 && K > 0, "gemm_bf16: bad sizes M=%d N=%d K=%d", M, N, K);
     QI_REQUIRE(K % 8 == 0, "gemm_bf16: K=%d must be a multiple of 8 (16-byte rows for TMA)", K);
     QI_REQUIRE(((uintptr_t)x & 15) == 0 && ((uintptr_t)w & 15) == 0, "gemm_bf16: operands must be 16-byte aligned");
     QI_REQUIRE(splits >= 1 && (splits == 1 || workspace), "gemm_bf16: split-K needs a workspace");
     QI_REQUIRE(out_dtype == qi::kF32 || out_dtype == qi::kBF16, "gemm_bf16: output type must be float32 or bfloat16");
-    QI_REQUIRE(epilogue == 0 || (epilogue == 1 && splits == 1 && out_dtype == qi::kBF16 && N % 2 == 0 && out),
+    QI_REQUIRE(epilogue == 0 || ((epilogue == 1 || epilogue == 3) && splits == 1 && out_dtype == qi::kBF16 && N % 2 == 0 && out),
                "gemm_bf16: the fused activation needs bfloat16 output, an even N and no K split");
+    RopeEpilogue glu{};
+    glu.limit = limit; glu.alpha = alpha;
     const int kb_total = (K + BK - 1) / BK;
     const int kb_per_split = (kb_total + splits - 1) / splits;
     QI_REQUIRE((splits - 1) * kb_per_split < kb_total, "gemm_bf16: %d splits leave one without work (K=%d)", splits, K);
     if (swap == 2) {
         // pairs of CTAs: tokens on the rows, no K split
         CUtensorMap pa, pb;
-        if (make_map(&pa, x, M, K, BM)) return 1;
+        if (make_map(&pa, x, M, K, BM, ldx)) return 1;
         if (make_map(&pb, w, N, K, BM)) return 1;
         if (splits > 1) {
             float* ws = (float*)workspace;
@@ -1147,6 +1166,7 @@ extern "C" int qi_gemm_bf16(const void* x, const void* w, void* out, int out_dty
             return 0;
         }
         if (epilogue == 1) return launch_pair<qi::bf16, 1>(pa, pb, (qi::bf16*)out, M, N, K, N / 2, status, stream);
+        if (epilogue == 3) return launch_pair<qi::bf16, 3>(pa, pb, (qi::bf16*)out, M, N, K, N / 2, status, stream, glu);
         if (out_dtype == qi::kF32) return launch_pair<float, 0>(pa, pb, (float*)out, M, N, K, N, status, stream);
         return launch_pair<qi::bf16, 0>(pa, pb, (qi::bf16*)out, M, N, K, N, status, stream);
     }
@@ -1155,8 +1175,8 @@ extern "C" int qi_gemm_bf16(const void* x, const void* w, void* out, int out_dty
     const int rows_a = swap ? N : M, rows_b = swap ? M : N;
     QI_REQUIRE((long long)((rows_a + BM - 1) / BM) * ((rows_b + bn - 1) / bn) * splits < 2147483647LL, "gemm_bf16: too many tiles");
     CUtensorMap ma, mb;
-    if (make_map(&ma, a, rows_a, K, BM)) return 1;
-    if (make_map(&mb, b, rows_b, K, bn)) return 1;
+    if (make_map(&ma, a, rows_a, K, BM, swap ? 0 : ldx)) return 1;
+    if (make_map(&mb, b, rows_b, K, bn, swap ? ldx : 0)) return 1;
     const long long split_stride = (long long)M * N;
     int rc;
     if (splits > 1) {
@@ -1176,11 +1196,21 @@ extern "C" int qi_gemm_bf16(const void* x, const void* w, void* out, int out_dty
     if (epilogue == 1)
         return swap ? launch_bn<true, qi::bf16, 1>(bn, ma, mb, (qi::bf16*)out, rows_a, rows_b, K, N / 2, 1, kb_per_split, 0, status, stream)
                     : launch_bn<false, qi::bf16, 1>(bn, ma, mb, (qi::bf16*)out, rows_a, rows_b, K, N / 2, 1, kb_per_split, 0, status, stream);
+    if (epilogue == 3)
+        return swap ? launch_bn<true, qi::bf16, 3>(bn, ma, mb, (qi::bf16*)out, rows_a, rows_b, K, N / 2, 1, kb_per_split, 0, status, stream, glu)
+                    : launch_bn<false, qi::bf16, 3>(bn, ma, mb, (qi::bf16*)out, rows_a, rows_b, K, N / 2, 1, kb_per_split, 0, status, stream, glu);
     if (out_dtype == qi::kF32)
         return swap ? launch_bn<true, float>(bn, ma, mb, (float*)out, rows_a, rows_b, K, N, 1, kb_per_split, 0, status, stream)
                     : launch_bn<false, float>(bn, ma, mb, (float*)out, rows_a, rows_b, K, N, 1, kb_per_split, 0, status, stream);
     return swap ? launch_bn<true, qi::bf16>(bn, ma, mb, (qi::bf16*)out, rows_a, rows_b, K, N, 1, kb_per_split, 0, status, stream)
                 : launch_bn<false, qi::bf16>(bn, ma, mb, (qi::bf16*)out, rows_a, rows_b, K, N, 1, kb_per_split, 0, status, stream);
+}
+
+extern "C" int qi_gemm_bf16(const void* x, const void* w, void* out, int out_dtype, int M, int N, int K,
+                            int swap, int bn, int splits, int epilogue, void* workspace, int* status,
+                            cudaStream_t stream) {
+    QI_REQUIRE(epilogue == 0 || epilogue == 1, "gemm_bf16: unknown epilogue %d", epilogue);
+    return qi_gemm_bf16_ex(x, 0, w, out, out_dtype, M, N, K, swap, bn, splits, epilogue, 0.f, 0.f, workspace, status, stream);
 }
 
 // The q/k/v projection of many tokens with what follows it fused into the epilogue:

@@ -454,7 +454,7 @@ ssm_chain_kernel(float* __restrict__ seg_state, float* __restrict__ state, long 
 template <typename TZ, typename TO>
 __global__ void __launch_bounds__(256)
 gated_group_rmsnorm_kernel(const float* __restrict__ y, const TZ* __restrict__ z, long long ldz, const float* __restrict__ gain,
-                           float eps, TO* __restrict__ out, int width, int groups, int mode, float out_scale) {
+                           float eps, TO* __restrict__ out, long long ldo, int width, int groups, int mode, float out_scale) {
     __shared__ float scratch[32];
     qi::pdl_wait();
     const int t = blockIdx.x, grp = blockIdx.y;
@@ -481,7 +481,7 @@ gated_group_rmsnorm_kernel(const float* __restrict__ y, const TZ* __restrict__ z
         if (mode == 1) v *= zz * sg;
         else if (mode == 2) v *= sg;
         else if (mode == 3) v *= zz;
-        out[(size_t)t * width + (size_t)grp * gw + i] = qi::from_f32<TO>(v * out_scale);
+        out[(size_t)t * ldo + (size_t)grp * gw + i] = qi::from_f32<TO>(v * out_scale);
     }
 }
 
@@ -491,7 +491,7 @@ constexpr int kNarrowGroup = 256;
 template <typename TZ, typename TO>
 __global__ void __launch_bounds__(256)
 gated_narrow_group_rmsnorm_kernel(const float* __restrict__ y, const TZ* __restrict__ z, long long ldz, const float* __restrict__ gain,
-                                  float eps, TO* __restrict__ out, long long n_groups, int width, int groups, int mode, float out_scale) {
+                                  float eps, TO* __restrict__ out, long long ldo, long long n_groups, int width, int groups, int mode, float out_scale) {
     qi::pdl_wait();
     const long long g = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
     if (g >= n_groups) return;
@@ -522,7 +522,7 @@ gated_narrow_group_rmsnorm_kernel(const float* __restrict__ y, const TZ* __restr
             if (mode == 1) r *= zz[m] * sg;
             else if (mode == 2) r *= sg;
             else if (mode == 3) r *= zz[m];
-            out[t * width + (size_t)grp * gw + i] = qi::from_f32<TO>(r * out_scale);
+            out[t * ldo + (size_t)grp * gw + i] = qi::from_f32<TO>(r * out_scale);
         }
     }
 }
@@ -628,12 +628,12 @@ extern "C" int qi_ssm_chain(float* seg_state, float* state, long long state_stri
 }
 
 // y float32 [n, width]; z [n, >= width] in z_dtype with `ldz` elements a row; gain float32 [width]; out [n, width] in out_dtype.
-// mode 0: rmsnorm_groups(y * silu(z)) * gain; 1: rmsnorm_groups(y) * gain * silu(z); 2: ... * sigmoid(z); 3: ... * z.
-extern "C" int qi_group_rmsnorm_gate(const float* y, const void* z, int z_dtype, long long ldz, const float* gain, float eps,
-                                     void* out, int out_dtype, int n, int width, int groups, int mode, float out_scale,
+// `ldo`: elements from one row of out to the next. mode 0: rmsnorm_groups(y * silu(z)) * gain; 1: rmsnorm_groups(y) * gain * silu(z); 2: ... * sigmoid(z); 3: ... * z.
+extern "C" int qi_group_rmsnorm_gate_ex(const float* y, const void* z, int z_dtype, long long ldz, const float* gain, float eps,
+                                     void* out, long long ldo, int out_dtype, int n, int width, int groups, int mode, float out_scale,
                                      cudaStream_t stream) {
     QI_REQUIRE(n >= 0 && width > 0 && groups > 0 && width % groups == 0, "gated_group_rmsnorm: bad sizes n=%d width=%d groups=%d", n, width, groups);
-    QI_REQUIRE(ldz >= width && groups <= 65535, "gated_group_rmsnorm: bad layout");
+    QI_REQUIRE(ldz >= width && ldo >= width && groups <= 65535, "gated_group_rmsnorm: bad layout");
     QI_REQUIRE(mode >= 0 && mode <= 3, "gated_group_rmsnorm: unknown mode %d", mode);
     if (n == 0) return 0;
     const long long n_groups = (long long)n * groups;
@@ -642,13 +642,19 @@ extern "C" int qi_group_rmsnorm_gate(const float* y, const void* z, int z_dtype,
         QI_DISPATCH_DTYPE(out_dtype, TO, {
             if (narrow)
                 qi::launch(gated_narrow_group_rmsnorm_kernel<TZ, TO>, dim3((unsigned)((n_groups + 7) / 8)), dim3(256), 0, stream, y,
-                           (const TZ*)z, ldz, gain, eps, (TO*)out, n_groups, width, groups, mode, out_scale);
+                           (const TZ*)z, ldz, gain, eps, (TO*)out, ldo, n_groups, width, groups, mode, out_scale);
             else
                 qi::launch(gated_group_rmsnorm_kernel<TZ, TO>, dim3(n, groups), dim3(256), 0, stream, y, (const TZ*)z, ldz, gain, eps,
-                           (TO*)out, width, groups, mode, out_scale);
+                           (TO*)out, ldo, width, groups, mode, out_scale);
         });
     });
     return qi::check_launch("gated_group_rmsnorm");
+}
+
+extern "C" int qi_group_rmsnorm_gate(const float* y, const void* z, int z_dtype, long long ldz, const float* gain, float eps,
+                                     void* out, int out_dtype, int n, int width, int groups, int mode, float out_scale,
+                                     cudaStream_t stream) {
+    return qi_group_rmsnorm_gate_ex(y, z, z_dtype, ldz, gain, eps, out, width, out_dtype, n, width, groups, mode, out_scale, stream);
 }
 
 extern "C" int qi_gated_group_rmsnorm(const float* y, const void* z, int z_dtype, long long ldz, const float* gain, float eps,

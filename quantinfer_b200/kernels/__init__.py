@@ -25,7 +25,7 @@ STATUS_NON_FINITE = 4
 STATUS_WAIT_TIMEOUT = 8
 STATUS_BAD_RANGE = 16
 
-ABI_VERSION = 14
+ABI_VERSION = 15
 
 
 def status_names(code: int) -> list:
@@ -450,6 +450,13 @@ def qk_norm_rope_kv(qkv, q_out, q_gain, k_gain, eps, cos, sin, rotary_dim, posit
 # attention
 
 
+def _req_out(out, name: str, dtype, rows: int, cols: int) -> int:
+    """An output [rows, cols] that may be a block of columns of wider rows; returns its row stride."""
+    if not isinstance(out, torch.Tensor) or not out.is_cuda or out.dtype != dtype or tuple(out.shape) != (rows, cols) or out.stride(1) != 1:
+        raise KernelError(f"{name}: out must be a CUDA tensor [{rows}, {cols}] of {dtype} with contiguous rows")
+    return out.stride(0) if rows > 1 else max(out.stride(0), cols)
+
+
 def _req_bias(bias, nq: int) -> None:
     """A distance bias of the attention kernels: float32 [nq, reach], reach >= 1."""
     if bias is not None:
@@ -470,7 +477,6 @@ def attention_generic(q, out, k_pages, v_pages, block_table, positions, token_re
     positions back adds bias[h, min(n, reach - 1)] to its score (after the cap)."""
     _req_bias(bias, nq)
     _req(q, "q", ndim=2)
-    _req(out, "out", q.dtype, 2)
     _req(k_pages, "k_pages", q.dtype, 4)
     _req(v_pages, "v_pages", q.dtype, 4)
     _req(block_table, "block_table", torch.int32, 2)
@@ -480,6 +486,7 @@ def attention_generic(q, out, k_pages, v_pages, block_table, positions, token_re
     dv = v_pages.shape[3]
     if q.shape[1] != nq * d or tuple(out.shape) != (n, nq * dv):
         raise KernelError(f"attention: q {tuple(q.shape)} / out {tuple(out.shape)} do not match {nq} heads of {d} / {dv}")
+    ldo = _req_out(out, "attention", q.dtype, n, nq * dv)
     if k_pages.shape[1] != nkv or k_pages.shape[3] != d or k_pages.shape[:3] != v_pages.shape[:3]:
         raise KernelError(f"attention: pages {tuple(k_pages.shape)} / {tuple(v_pages.shape)} do not match {nkv} kv heads of {d}")
     ldg = 0
@@ -495,7 +502,7 @@ def attention_generic(q, out, k_pages, v_pages, block_table, positions, token_re
           _ptr(q), _ptr(out), _code(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
         block_table.shape[1], k_pages.shape[2], k_pages.shape[0], _ptr(positions), _ptr(token_req), n,
         nq, nkv, d, dv, C.c_float(scale), C.c_float(softcap or 0.0), C.c_float(out_scale), int(window or 0), int(chunk or 0), _ptr(gate), C.c_longlong(ldg), _ptr(sink),
-        _ptr(bias), bias.shape[1] if bias is not None else 0, _ptr(status), _stream())
+        _ptr(bias), bias.shape[1] if bias is not None else 0, C.c_longlong(ldo), _ptr(status), _stream())
 
 
 def attention_mma_supported(nq: int, nkv: int, d: int) -> bool:
@@ -563,7 +570,7 @@ def attention_prefill(q, out, k_pages, v_pages, block_table, q_start, start_pos,
     if impl is None and use_tma is not None:
         impl = "tma" if use_tma else "cpasync"
     _req(q, "q", torch.bfloat16, 2)
-    _req(out, "out", torch.bfloat16, 2)
+    ldo = _req_out(out, "attention_prefill", torch.bfloat16, q.shape[0], nq * d)
     _req(k_pages, "k_pages", torch.bfloat16, 4)
     _req(v_pages, "v_pages", torch.bfloat16, 4)
     for t, name in ((block_table, "block_table"), (q_start, "q_start"), (start_pos, "start_pos"),
@@ -599,10 +606,11 @@ def attention_prefill(q, out, k_pages, v_pages, block_table, q_start, start_pos,
             k_pages.shape[2], k_pages.shape[0], _ptr(q_start), _ptr(start_pos), _ptr(tile_req), _ptr(tile_q0),
             tile_req.numel(), q.shape[0], nq, nkv, d, C.c_float(scale), int(window or 0), int(chunk or 0), _ptr(gate),
             C.c_longlong(ldg), ranges, _ptr(ws), _ptr(status), C.c_float(softcap or 0.0), C.c_float(out_scale), _ptr(sink),
-            _ptr(bias), bias.shape[1] if bias is not None else 0, _stream())
+            _ptr(bias), bias.shape[1] if bias is not None else 0, C.c_longlong(ldo), _stream())
         return
     if chunk or gate is not None or softcap or out_scale != 1.0 or sink is not None or bias is not None:
         raise KernelError(f"attention_prefill: the {impl!r} kernel takes neither a chunk bound, a gate, a soft cap, an output factor, a sink nor a bias")
+    _req(out, "out", torch.bfloat16, 2)
     if impl not in ("tma", "cpasync"):
         raise KernelError(f"attention_prefill: unknown kernel {impl!r}")
     if impl == "tma":
@@ -907,23 +915,24 @@ _plans = {}
 
 
 def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out, plan=None, status=None, epilogue: str | None = None,
-              keep_partials: bool = False):
+              keep_partials: bool = False, glu=None):
     """out[M, N] = x[M, K] @ w[N, K]^T on the tcgen05 tensor cores; x, w bfloat16; out
     bfloat16 or float32. `plan` = (orientation, tile width, splits) overrides the choice.
 
     epilogue="silu_mul": w's rows are (gate, up) pairs and out is [M, N / 2] =
-    silu(gate) * up. keep_partials=True: when the plan splits K, the float32 partial sums
+    silu(gate) * up; "glu_clamped" with `glu` = (limit, alpha): g sigmoid(alpha g) (u + 1), g = min(gate, limit), u =
+    clamp(up, -limit, limit). x may be a block of columns of wider rows (a multiple of 8 elements apart). keep_partials=True: when the plan splits K, the float32 partial sums
     [splits, M, N] are returned unreduced (and `out` is not written); else `out` is returned."""
-    _req(x, "x", torch.bfloat16, 2)
+    _cols(x, "x", torch.bfloat16)
     _req(w, "w", torch.bfloat16, 2)
     M, K = x.shape
     N = w.shape[0]
-    if epilogue not in (None, "silu_mul"):
+    if epilogue not in (None, "silu_mul", "glu_clamped") or (epilogue == "glu_clamped") != (glu is not None):
         raise KernelError(f"gemm_bf16: unknown epilogue {epilogue!r}")
     swap, bn, splits = plan if plan is not None else gemm_bf16_plan(M, N, K, allow_split=epilogue is None)
     epi = 0
-    if epilogue == "silu_mul":
-        epi, splits = 1, 1
+    if epilogue is not None:
+        epi, splits = (1 if epilogue == "silu_mul" else 3), 1
     n_out = N // 2 if epi else N
     partial_only = keep_partials and splits > 1
     if not partial_only:
@@ -935,10 +944,10 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out, plan=None, status=None, epi
         status = _gemm_status.get(x.device)
         if status is None:
             status = _gemm_status[x.device] = torch.zeros(1, dtype=torch.int32, device=x.device)
-    _call('gemm', "gemm_bf16", library().qi_gemm_bf16,
-          _ptr(x), _ptr(w), _ptr(None if partial_only else out),
+    _call('gemm', "gemm_bf16", library().qi_gemm_bf16_ex,
+          _ptr(x), C.c_longlong(x.stride(0) if M > 1 else 0), _ptr(w), _ptr(None if partial_only else out),
                                 BF16 if partial_only else _code(out), M, N, K, int(swap), bn, splits, epi,
-                                _ptr(ws), _ptr(status), _stream())
+                                C.c_float(glu[0] if glu else 0.0), C.c_float(glu[1] if glu else 0.0), _ptr(ws), _ptr(status), _stream())
     return ws if partial_only else out
 
 
@@ -1357,19 +1366,19 @@ def gated_group_rmsnorm(y, z, gain, eps: float, out, groups: int, gate: str = "s
     """Every width / groups coordinates of a row by their own root mean square, a gain, and a gate z:
     "silu_before": rmsnorm_groups(y * silu(z)) * gain; "silu": rmsnorm_groups(y) * gain * silu(z); "sigmoid": ... * sigmoid(z);
     "plain": ... * z. `out_scale` multiplies the result.
-    y float32 [n, width]; z [n, width] (may be a block of columns of wider rows); gain float32 [width]."""
+    y float32 [n, width]; z and out [n, width] (may be blocks of columns of wider rows); gain float32 [width]."""
     if gate not in GATE_MODES:
         raise KernelError(f"gated_group_rmsnorm: gate {gate!r} is not known (one of {sorted(GATE_MODES)})")
     _req(y, "y", torch.float32, 2)
     if not z.is_cuda or z.dim() != 2 or z.stride(1) != 1 or z.shape != y.shape:
         raise KernelError("gated_group_rmsnorm: z must match y, with contiguous rows")
     _req(gain, "gain", torch.float32, 1)
-    _req(out, "out", ndim=2)
     n, width = y.shape
-    if gain.numel() != width or out.shape != y.shape or groups <= 0 or width % groups:
+    ldo = _req_out(out, "gated_group_rmsnorm", out.dtype, n, width)
+    if gain.numel() != width or groups <= 0 or width % groups:
         raise KernelError("gated_group_rmsnorm: shapes do not agree")
-    _call("norm", "gated_group_rmsnorm", library().qi_group_rmsnorm_gate, _ptr(y), _ptr(z), _code(z), C.c_longlong(z.stride(0)),
-          _ptr(gain), C.c_float(eps), _ptr(out), _code(out), n, width, groups, GATE_MODES[gate], C.c_float(out_scale), _stream())
+    _call("norm", "gated_group_rmsnorm", library().qi_group_rmsnorm_gate_ex, _ptr(y), _ptr(z), _code(z), C.c_longlong(z.stride(0)),
+          _ptr(gain), C.c_float(eps), _ptr(out), C.c_longlong(ldo), _code(out), n, width, groups, GATE_MODES[gate], C.c_float(out_scale), _stream())
 
 
 # --------------------------------------------------------------------------
@@ -1671,6 +1680,7 @@ class _LeadRows:
     def __init__(self, batch, lead: int):
         self.q_start, self.start_pos, self.n_requests = batch.q_start[:lead + 1], batch.start_pos[:lead], lead
         self.positions, self.token_req = batch.positions[:lead], batch.token_req[:lead]
+        self.all_decode, self.max_kv_len = True, batch.max_kv_len
 
 
 def gated_attention_mma_supported(nq: int, nkv: int, d: int, dv: int) -> bool:
@@ -1680,7 +1690,7 @@ def gated_attention_mma_supported(nq: int, nkv: int, d: int, dv: int) -> bool:
 
 def gated_attention(q, out, k_pages, v_pages, block_table, batch, nq, nkv, d, dv, scale: float, window: int, chunk: int, gate,
                     status, impl: str | None = None, softcap: float = 0.0, out_scale: float = 1.0, sink=None,
-                    key_ranges: int | None = None, bias=None) -> None:
+                    key_ranges: int | None = None, bias=None, grouped_heads: bool | None = None) -> None:
     """Attention with separate key and value sizes, an optional chunk bound and an optional output gate, by the
     kernel that fits: "mma" (bfloat16, head sizes that are multiples of 8 up to 128: flash form on the tensor
     cores, tiles found on the device from the step's arrays) or "generic" (32-bit arithmetic, any sizes). A step
@@ -1691,7 +1701,8 @@ def gated_attention(q, out, k_pages, v_pages, block_table, batch, nq, nkv, d, dv
     [nq, reach]: a key n positions back adds bias[h, min(n, reach - 1)] to its score). A step of single tokens on
     "mma" cuts every token's keys into `key_ranges` ranges over separate CTAs (None: as many as fill the device, from
     the longest context and the window, so that a captured step serves its whole context bucket) and adds the parts
-    in a second kernel."""
+    in a second kernel; there the query heads that share a key head are the rows of one tile where there are at most 16
+    of them (`grouped_heads` forces either form). `out` may be a block of columns of wider rows."""
     if impl is None and q.dtype == torch.bfloat16 and d == dv and not batch.all_decode and batch.tile_req.numel() and (
             gate is None or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)) and attention_prefill_tcgen05_supported(
             nq, nkv, d, k_pages.shape[2], block_table.shape[1]):
@@ -1718,11 +1729,11 @@ def gated_attention(q, out, k_pages, v_pages, block_table, batch, nq, nkv, d, dv
         if sink.numel() != nq:
             raise KernelError("gated_attention: one sink a query head")
     _req(q, "q", torch.bfloat16, 2)
-    _req(out, "out", torch.bfloat16, 2)
     _req(k_pages, "k_pages", torch.bfloat16, 4)
     _req(v_pages, "v_pages", torch.bfloat16, 4)
     _req(block_table, "block_table", torch.int32, 2)
     n = q.shape[0]
+    ldo = _req_out(out, "gated_attention", torch.bfloat16, n, nq * dv)
     if q.shape[1] != nq * d or tuple(out.shape) != (n, nq * dv):
         raise KernelError(f"gated_attention: q {tuple(q.shape)} / out {tuple(out.shape)} do not match {nq} heads of {d} / {dv}")
     if tuple(k_pages.shape[1:]) != (nkv, k_pages.shape[2], d) or tuple(v_pages.shape) != (k_pages.shape[0], nkv, k_pages.shape[2], dv):
@@ -1732,10 +1743,11 @@ def gated_attention(q, out, k_pages, v_pages, block_table, batch, nq, nkv, d, dv
         if not gate.is_cuda or gate.dtype != q.dtype or gate.dim() != 2 or gate.stride(1) != 1 or gate.shape != out.shape:
             raise KernelError("gated_attention: the gate must be [n, nq dv] in q's type with contiguous rows")
         ldg = gate.stride(0)
-    ranges, ws = 1, None
+    ranges, ws, grouped = 1, None, False
     if getattr(batch, "all_decode", False) and n <= 65535:
+        grouped = (nq // nkv <= 16) if grouped_heads is None else grouped_heads
         keys = min(window or batch.max_kv_len, chunk or batch.max_kv_len, batch.max_kv_len)
-        ranges = key_ranges or max(1, min(-(-keys // 128), 296 // max(n * nq, 1), 64))
+        ranges = key_ranges or max(1, min(-(-keys // 128), 296 // max(n * (nkv if grouped else nq), 1), 64))
         if ranges > 1:
             ws = torch.empty(n * nq * ranges * (dv + 2), dtype=torch.float32, device=q.device)
     _call("attention", "gated_attention_mma", library().qi_gated_attention_mma_bias, _ptr(q), _ptr(out), _ptr(k_pages), _ptr(v_pages),
@@ -1743,4 +1755,4 @@ def gated_attention(q, out, k_pages, v_pages, block_table, batch, nq, nkv, d, dv
           batch.n_requests, n, nq, nkv, d, dv, C.c_float(scale), C.c_float(softcap or 0.0), C.c_float(out_scale), int(window or 0),
           int(chunk or 0), _ptr(gate), C.c_longlong(ldg), _ptr(sink),
           _ptr(bias), bias.shape[1] if bias is not None else 0, ranges, _ptr(ws),
-          _ptr(status), _stream())
+          int(grouped), C.c_longlong(ldo), _ptr(status), _stream())

@@ -328,8 +328,9 @@ class HyperBlock(Part):
         self.mixer = build_part("mixer", spec.mixer, runtime)
         self.ffn = build_part("ffn", spec.ffn, runtime) if spec.ffn is not None else None
         self.ffn_norm = build_part("norm", spec.ffn_norm, runtime) if spec.ffn is not None else None
-        if hasattr(self.mixer, "keep_partials"):
-            self.mixer.keep_partials = True       # the streams' kernel adds a split product's partial sums itself
+        for p in (self.mixer, self.ffn):
+            if hasattr(p, "keep_partials"):
+                p.keep_partials = True            # the streams' kernel adds a split product's partial sums itself
         self.read, self.share, self.mix = [], [], []
         self._parts = tuple(p for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.ffn) if p is not None)
 

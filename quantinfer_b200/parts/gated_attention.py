@@ -135,29 +135,33 @@ class GatedAttention(Part):
         return StateNeed((self.taps - 1, self.qkv_cols), torch.float32)
 
     def forward(self, x, batch, cache):
+        out = torch.empty((x.shape[0], self.H * self.dv), dtype=x.dtype, device=x.device)
+        self.mix(self.proj(x), batch, cache, out)
+        return self.o(out, keep_partials=True)
+
+    def mix(self, proj, batch, cache, out, out_scale: float = 1.0):
+        """From the projected rows (`proj`, maybe a block of columns of wider rows) to what the output projection reads, times
+        `out_scale`, written to `out` [n, heads value_dim] (likewise)."""
         rt, s = self.runtime, self.spec
-        n = x.shape[0]
+        n = proj.shape[0]
         table = batch.block_tables[cache.group]
-        proj = self.proj(x)
         if self.taps is not None:
-            conved = torch.empty((n, self.qkv_cols), dtype=x.dtype, device=x.device)
+            conved = torch.empty((n, self.qkv_cols), dtype=proj.dtype, device=proj.device)
             kernels.short_conv(proj[:, :self.qkv_cols], self.conv_w, cache.mixer_state, [conved], None, batch.token_req, batch.q_start,
                                batch.start_pos, batch.slot_ids, residual=False)
             gate_src, proj = proj, conved
         else:
             gate_src = proj
-        q = torch.empty((n, self.H * self.d), dtype=x.dtype, device=x.device)
+        q = torch.empty((n, self.H * self.d), dtype=proj.dtype, device=proj.device)
         kernels.bias_rope_kv(proj, self.bias, q, self.inv_freq, self.rot, self.interleaved, batch.positions, batch.token_req,
                              table, cache.page_size, cache.k_pages if cache.writes else None,
                              cache.v_pages if cache.writes else None, self.H, self.G, self.d, self.dv, rt.status,
                              q_gain=self.q_gain, k_gain=self.k_gain, norm_eps=getattr(s, "qk_norm_eps", 0.0),
                              values_from_keys=self.v_from_k, head_norm=self.qk_norm == "head", q_temp=self.q_temp)
-        out = torch.empty((n, self.H * self.dv), dtype=x.dtype, device=x.device)
-        gate = gate_src[:, self.qkv_cols:] if s.out_gate else None
+        gate = gate_src[:, self.qkv_cols:self.qkv_cols + self.H * self.dv] if s.out_gate else None
         kernels.gated_attention(q, out, cache.k_pages, cache.v_pages, table, batch, self.H, self.G, self.d, self.dv, s.scale,
                                 s.window or 0, s.chunk or 0, gate, rt.status, softcap=getattr(s, "softcap", None) or 0.0,
-                                out_scale=getattr(s, "out_scale", 1.0), sink=self.sink, bias=self.dist_bias)
-        return self.o(out, keep_partials=True)
+                                out_scale=out_scale * getattr(s, "out_scale", 1.0), sink=self.sink, bias=self.dist_bias)
 
 
 register_part("mixer", "gated_attention", GatedAttention)

@@ -48,12 +48,14 @@ class Linear:
         [splits, tokens, out] of a K-split product, for a consumer that adds them itself
         (the fused add + norm does)."""
         out_dtype = out_dtype or x.dtype
+        if not x.is_contiguous() and (x.stride(1) != 1 or x.stride(0) % 8 or x.data_ptr() % 16):
+            x = x.contiguous()            # (a block of columns on 16-byte boundaries is read where it lies)
         out = torch.empty((x.shape[0], self.out_features), dtype=out_dtype, device=x.device)
         if x.shape[0] == 0:
             return out
         if self.tensor_core(x, out_dtype):
             return kernels.gemm_bf16(x, self.weight, out, status=self.runtime.status, keep_partials=keep_partials)
-        kernels.gemm_simt(x, self.weight, out)
+        kernels.gemm_simt(x if x.is_contiguous() else x.contiguous(), self.weight, out)
         return out
 
     def forward_act_mul(self, x: torch.Tensor, activation: str = "silu") -> torch.Tensor:
@@ -69,6 +71,18 @@ class Linear:
             return act
         gu = self.forward(x)
         kernels.act_mul(gu, act, activation, interleaved=True)
+        return act
+
+    def forward_glu_clamped(self, x: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+        """g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit), of a projection whose weight
+        rows are (gate, up) pairs: [tokens, out / 2]; in the tensor-core product's epilogue, or by a kernel over its output."""
+        act = torch.empty((x.shape[0], self.out_features // 2), dtype=x.dtype, device=x.device)
+        if x.shape[0] == 0:
+            return act
+        if self.tensor_core(x, x.dtype):
+            kernels.gemm_bf16(x, self.weight, act, status=self.runtime.status, epilogue="glu_clamped", glu=(limit, alpha))
+        else:
+            kernels.glu_clamped(self.forward(x), act, limit, alpha, interleaved=True)
         return act
 
     def forward_silu_mul(self, x: torch.Tensor) -> torch.Tensor:

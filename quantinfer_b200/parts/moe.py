@@ -36,6 +36,7 @@ class ClampedGLU(Part):
         h, i = spec.hidden_size, spec.intermediate_size
         self.gate_up = Linear(runtime, 2 * i, h, spec.prefix + "gate+up")
         self.down = Linear(runtime, h, i, spec.prefix + "down")
+        self.keep_partials = False        # True: the block's next norm adds a split product's partial sums itself
 
     @classmethod
     def needs_of_spec(cls, spec):
@@ -47,14 +48,11 @@ class ClampedGLU(Part):
         g, u = tensors[p + "gate"], tensors[p + "up"]
         if g.dtype != u.dtype:
             g, u = g.to(torch.float32), u.to(torch.float32)
-        self.gate_up.load(torch.cat([g, u], dim=0))
+        self.gate_up.load(torch.stack([g, u], dim=1).reshape(2 * g.shape[0], g.shape[1]))     # rows in (gate, up) pairs
         self.down.load(tensors[p + "down"])
 
     def forward(self, x):
-        gu = self.gate_up(x)
-        a = torch.empty((x.shape[0], self.spec.intermediate_size), dtype=x.dtype, device=x.device)
-        kernels.glu_clamped(gu, a, self.spec.limit, self.spec.alpha)
-        return self.down(a)
+        return self.down(self.gate_up.forward_glu_clamped(x, self.spec.limit, self.spec.alpha), keep_partials=self.keep_partials)
 
     __call__ = forward
 
