@@ -13,7 +13,8 @@ group, cut into pages of `page_size` positions:
 * a request has, per group, a *block table*: `table[b]` is the page that holds
   positions `b * page_size ... (b + 1) * page_size - 1`, or -1.
 * groups with a window give pages back as soon as every position in them lies
-  outside the window of all coming queries; all pages go back when the request
+  outside the window of all coming queries (pages that hold positions a need
+  keeps visible from the sequence's start are never given back that way); all pages go back when the request
   closes, and a step that fails gives back what it took (`rollback`).
 * a *slot* is a request's index into per-request arrays of fixed size: mixer
   state (`StateNeed` entries, `[num_slots, *shape]`, zeroed at `open`) and
@@ -193,7 +194,8 @@ class CacheManager:
         w = self.groups[group].need.window
         c = getattr(self.groups[group].need, "chunk", None)
         live = length if w is None else min(length, w)
-        return live if not c else min(live, length - (length - 1) // c * c if length else 0)
+        live = live if not c else min(live, length - (length - 1) // c * c if length else 0)
+        return min(length, live + getattr(self.groups[group].need, "keep_first", 0))
 
     # ---- requests -------------------------------------------------------
 
@@ -262,7 +264,8 @@ class CacheManager:
             if chunk:
                 first_needed = max(first_needed, rc.length // chunk * chunk)
             table = rc.tables[gi]
-            for b in range(min(first_needed // self.page_size, len(table))):
+            kept = -(-getattr(g.need, "keep_first", 0) // self.page_size)      # pages that hold kept first positions
+            for b in range(kept, min(first_needed // self.page_size, len(table))):
                 if table[b] >= 0:
                     g.allocator.free(table[b])
                     table[b] = -1

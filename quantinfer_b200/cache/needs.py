@@ -12,13 +12,15 @@ class PagedKVNeed:
     positions, in pages [num_pages, num_kv_heads, page_size, head_dim] (values
     [..., value_dim] when that is given). `chunk`: queries see only the keys of
     their own chunk of that many positions (counted from the sequence's start),
-    so the pages of earlier chunks go back as soon as a request has passed them."""
+    so the pages of earlier chunks go back as soon as a request has passed them. `keep_first`:
+    the first positions of a sequence stay visible behind a window or chunk, so their pages stay."""
 
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     value_dim: Optional[int] = None
     chunk: Optional[int] = None
+    keep_first: int = 0
 
     def pools(self, page_size: int) -> tuple:
         """Shapes of a page in the key pool and in the value pool."""
@@ -32,7 +34,8 @@ class PagedKVNeed:
             return None
         if self.chunk != other.chunk:      # readers with other chunks: keep what any of them may see
             return PagedKVNeed(self.num_kv_heads, self.head_dim, None, self.value_dim, None)
-        return PagedKVNeed(self.num_kv_heads, self.head_dim, _wider(self.window, other.window), self.value_dim, self.chunk)
+        return PagedKVNeed(self.num_kv_heads, self.head_dim, _wider(self.window, other.window), self.value_dim, self.chunk,
+                           max(self.keep_first, other.keep_first))
 
 
 @dataclass(frozen=True)

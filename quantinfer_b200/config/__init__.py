@@ -6,6 +6,7 @@ from .kiruvik import KiruvikConfig
 from .dulotar import DulotarConfig
 from .lemotar import LemotarConfig
 from .siditar import SiditarConfig
+from .bomipel import BomipelConfig
 from .spec import (AttentionSpec, BigramEmbeddingSpec, DenseFeedForwardSpec, EmbeddingSpec, FeedForwardSpec, HeadSpec,
                    LatentAttentionSpec, LayerCall, LayerSpec, ModelSpec, NormSpec, ParallelLayerSpec, PositionSpec,
                    RotarySpec, ShortConvSpec, ClampedGLUSpec, GatedAttentionSpec, MoESpec, ReentrySpec, SandwichLayerSpec,
@@ -20,5 +21,5 @@ __all__ = [
     "KiruvikConfig", "ClampedGLUSpec", "GatedAttentionSpec", "MoESpec", "ReentrySpec", "SandwichLayerSpec", "StateSpaceSpec",
     "DulotarConfig", "ConvPreNormLayerSpec", "LightningAttentionSpec", "MinGRUSpec", "ParallelMixersSpec", "TimeMixSpec",
     "LemotarConfig", "GatedDeltaSpec", "PostNormLayerSpec",
-    "SiditarConfig", "GatedLinearAttentionSpec", "HyperLayerSpec", "StreamSumNormSpec",
+    "SiditarConfig", "GatedLinearAttentionSpec", "HyperLayerSpec", "StreamSumNormSpec", "BomipelConfig",
 ]

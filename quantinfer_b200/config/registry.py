@@ -85,6 +85,9 @@ def _register_builtin() -> None:
     from .siditar import ARCHITECTURE as SIDITAR, SiditarConfig
 
     register_architecture(SIDITAR, SiditarConfig)
+    from .bomipel import ARCHITECTURE as BOMIPEL, BomipelConfig
+
+    register_architecture(BOMIPEL, BomipelConfig)
 
 
 _register_builtin()

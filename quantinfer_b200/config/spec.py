@@ -25,7 +25,8 @@ class NormSpec:
     coordinates, the tensor named `prefix` itself, of shape []. "dyt": dynamic tanh, tanh(alpha x) w + b with no
     statistic of the row (eps unused): w is the tensor named `prefix` itself, b `prefix + ".b"`, alpha
     `prefix + ".alpha"` of shape []. "layernorm": (x - mean) / sqrt(variance + eps) * w + b with the variance the mean
-    squared deviation; w is the tensor named `prefix` itself, b `prefix + ".b"`. "layernorm_nobias": the same without b."""
+    squared deviation; w is the tensor named `prefix` itself, b `prefix + ".b"`. "layernorm_nobias": the same without b.
+    "rmsnorm_named": gain per coordinate, the tensor named `prefix` itself."""
 
     size: int
     eps: float
@@ -90,6 +91,9 @@ class RotarySpec:
                                       # `original` positions have their frequency divided by `factor`, pairs that turn
                                       # more than `fast` times keep it, a linear ramp over the pair's number lies
                                       # between (YaRN); cos and sin are then multiplied by 0.1 ln(factor) + 1
+    bands: Optional[tuple] = None     # (factor, low, high, original): a pair whose wavelength 2 pi / f is above original / low
+                                      # has its frequency divided by `factor`, one below original / high keeps it; between
+                                      # them (1 - s) f / factor + s f with s = (original / wavelength - low) / (high - low)
 
 
 @dataclass(frozen=True)
@@ -98,7 +102,8 @@ class LatentAttentionSpec:
     gain per coordinate) and a rotated key part of `rot_dim` numbers that all heads share; per head the
     key's plain part (`head_dim` numbers) and the value (`value_dim`) are projections of the latent.
     `shares_latent`: the layer has no latent projection and reads the cache entry of another layer.
-    `sink`: the softmax's denominator holds one more learned term per head."""
+    `sink`: the softmax's denominator holds one more learned term per head. `q_rank`: queries come through a latent of
+    their own, W_uq rmsnorm(W_dq x) (tensors `dq`, `dq.norm`, `uq` in the place of `q`)."""
 
     hidden_size: int
     num_heads: int
@@ -115,6 +120,7 @@ class LatentAttentionSpec:
     prefix: str = ""
     kind: str = "latent_attention"
     out_gate: bool = False            # the concatenated heads are multiplied by sigmoid(W_g x) (`g`) before the output projection
+    q_rank: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -146,7 +152,8 @@ class ParallelLayerSpec:
     """One block with one norm whose output feeds the mixer and the feed-forward side by side:
     h = norm(x); x += gate_m * mixer(conv_m(h)) + gate_f * ffn(conv_f(h)). `conv` (optional) is the bank
     of input convolutions, one filter per sublayer; `gate_names` (optional) are the prefixes of the sigmoid
-    gates' projections of h, one per sublayer ("<name>" the matrix, "<name>.b" the bias). `ffn` may be None."""
+    gates' projections of h, one per sublayer ("<name>" the matrix, "<name>.b" the bias). `ffn` may be None. `kind`
+    "parallel": neither gates nor convolutions, x += mixer(h) + ffn(h)."""
 
     norm: NormSpec
     mixer: object
@@ -215,6 +222,10 @@ class GatedAttentionSpec:
                                        # `q.norm`, `k.norm` [head_dim] that the heads share. "whole": q (all heads at once) and k (likewise) each pass one RMS norm over the whole
                                        # projection before the rotation, gains `q.norm` [heads head_dim], `k.norm`
     qk_norm_eps: float = 1e-6
+    keep_first: int = 0                # the sequence's first n keys stay visible behind the window or chunk, at their true positions
+    value_mix: Optional[str] = None    # "first": the layer's values (before any mixing) are what later layers of the same step mix in;
+                                       # "mix": values become (1 - a) v + a v_first before they are cached, a the tensor `vmix` of
+                                       # shape [] (which a "first" layer has too, unused)
 
 
 @dataclass(frozen=True)
@@ -412,19 +423,25 @@ class ClampedGLUSpec:
 
 @dataclass(frozen=True)
 class MoESpec:
-    """Mixture of `experts` small feed-forwards of the :class:`ClampedGLUSpec` form (`e<k>.gate` and so on), of which
-    a token uses `top`: scores = softmax of the router's logits over all experts (32-bit); the choice is by score +
-    `correction`, the weights are the chosen scores over their sum (+ 1e-20) times `router_scale`. `shared`
+    """Mixture of `experts` small feed-forwards (`e<k>.gate`, `.up`, `.down`; of the :class:`ClampedGLUSpec` form, or the
+    plain gated one of a :class:`FeedForwardSpec` with silu), of which a token uses `top`: scores = softmax of the router's
+    logits over all experts, or the sigmoid of each (`scoring`), in 32-bit; the choice is by score + `correction` (a tensor,
+    unless `has_correction` is off), the weights are the chosen scores over their sum (+ 1e-20), or as they are without
+    `normalize`, times `router_scale`. A weight multiplies its expert's output, or its input (`weight_on`). `shared`
     (optional) runs for every token and is added."""
 
     hidden_size: int
     experts: int
     top: int
     router_scale: float
-    expert: ClampedGLUSpec            # its prefix is the feed-forward's; expert k's tensors follow `e<k>.`
+    expert: object                    # its prefix is the feed-forward's; expert k's tensors follow `e<k>.`
     shared: Optional[ClampedGLUSpec] = None
     prefix: str = ""
     kind: str = "moe"
+    scoring: str = "softmax"          # or "sigmoid"
+    has_correction: bool = True
+    normalize: bool = True
+    weight_on: str = "output"         # or "input"
 
 
 @dataclass(frozen=True)

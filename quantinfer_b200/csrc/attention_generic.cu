@@ -8,7 +8,8 @@
 //     out     = sum_j softmax(score)_j * v_j
 // with lo = 0, or p - window + 1 for a windowed layer, or the start of p's chunk
 // (floor(p / chunk) * chunk, chunks counted from the sequence's first position)
-// for a chunked layer; both bounds may hold at once. A soft cap c replaces each
+// for a chunked layer; both bounds may hold at once, and the sequence's first `keep_first` keys may stay visible
+// whatever those bounds say. A soft cap c replaces each
 // score by c tanh(score / c) before the softmax; a distance bias then adds a number per
 // head that depends on p - j alone. Values may have another
 // size `dv` than queries and keys, and the result may be multiplied, element by
@@ -39,7 +40,7 @@ attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const T* 
                          const int* __restrict__ positions, const int* __restrict__ token_req,
                          int nq, int nkv, int d, int dv, float scale, float softcap, float out_scale, int window, int chunk,
                          const T* __restrict__ gate, long long ldg, const float* __restrict__ sink, const float* __restrict__ bias, int bias_len,
-                         long long ldo, int* __restrict__ status) {
+                         long long ldo, int keep_first, int* __restrict__ status) {
     extern __shared__ float smem[];
     float* q_s = smem;                          // [d]
     float* part_acc = smem + d;                 // [kWarps][dv]
@@ -55,6 +56,8 @@ attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const T* 
     const int* table = block_table + (size_t)r * max_blocks;
     int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
     if (chunk > 0) lo = max(lo, pos / chunk * chunk);
+    // the keys in one row of numbers: the kept first ones that lie before `lo`, then lo .. pos
+    const int head = min(keep_first, lo), last = head + pos - lo;
 
     const T* qrow = q + ((size_t)t * nq + h) * d;
     for (int i = threadIdx.x; i < d; i += blockDim.x) q_s[i] = qi::to_f32<T>(qrow[i]);
@@ -66,9 +69,9 @@ attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const T* 
     for (int i = 0; i < kAccPerLane; ++i) acc[i] = 0.f;
 
     bool bad_page = false;
-    for (int base = lo + warp * 32; base <= pos; base += kWarps * 32) {
-        const int j = base + lane;
-        const bool valid = j <= pos;
+    for (int base = warp * 32; base <= last; base += kWarps * 32) {
+        const int at = base + lane, j = at < head ? at : lo + at - head;
+        const bool valid = at <= last;
         float s = -INFINITY;
         if (valid) {
             const int page = table[j / page_size];
@@ -91,10 +94,10 @@ attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const T* 
         l = l * corr + qi::warp_sum(p);
 #pragma unroll
         for (int i = 0; i < kAccPerLane; ++i) acc[i] *= corr;
-        const int count = min(32, pos - base + 1);
+        const int count = min(32, last - base + 1);
         for (int jj = 0; jj < count; ++jj) {
             const float pj = __shfl_sync(0xffffffffu, p, jj);
-            const int key = base + jj;
+            const int key = base + jj < head ? base + jj : lo + base + jj - head;
             const int page = table[key / page_size];
             if (page < 0 || page >= num_pages) continue;
             const T* vrow = v_pages + (((size_t)page * nkv + hk) * page_size + (key % page_size)) * (size_t)dv;
@@ -147,14 +150,15 @@ attention_generic_kernel(const T* __restrict__ q, T* __restrict__ out, const T* 
 // softcap c > 0: a score s becomes c tanh(s / c) before the softmax (0: scores as they are); out_scale multiplies the result.
 // sink (may be null): float32 [nq]; the softmax's denominator of head h holds exp(sink[h]) once more.
 // bias (may be null): float32 [nq, bias_len]; a key n positions back adds bias[h, min(n, bias_len - 1)] to its score.
-// ldo: elements from one row of out to the next.
+// ldo: elements from one row of out to the next. keep_first: keys 0 .. keep_first - 1 stay visible behind a window or chunk.
 extern "C" int qi_attention_generic_bias(const void* q, void* out, int dtype, const void* k_pages,
                                        const void* v_pages, const int* block_table, int max_blocks,
                                        int page_size, int num_pages, const int* positions,
                                        const int* token_req, int n_tokens, int nq, int nkv, int d, int dv,
                                        float scale, float softcap, float out_scale, int window, int chunk, const void* gate,
-                                       long long ldg, const float* sink, const float* bias, int bias_len, long long ldo, int* status,
-                                       cudaStream_t stream) {
+                                       long long ldg, const float* sink, const float* bias, int bias_len, long long ldo,
+                                       int keep_first, int* status, cudaStream_t stream) {
+    QI_REQUIRE(keep_first >= 0, "attention: keep_first must be >= 0 (0 = none)");
     QI_REQUIRE(ldo >= (long long)nq * dv, "attention: the output's rows are too short");
     QI_REQUIRE(!bias || bias_len > 0, "attention: an empty distance bias");
     QI_REQUIRE(n_tokens >= 0 && nq > 0 && nkv > 0 && d > 0 && dv > 0, "attention: bad sizes");
@@ -176,7 +180,7 @@ extern "C" int qi_attention_generic_bias(const void* q, void* out, int dtype, co
                 (const T*)q + (size_t)t0 * nq * d, (T*)out + (size_t)t0 * ldo, (const T*)k_pages,
                 (const T*)v_pages, block_table, max_blocks, page_size, num_pages, positions + t0,
                 token_req + t0, nq, nkv, d, dv, scale, softcap, out_scale, window, chunk,
-                gate ? (const T*)gate + (size_t)t0 * ldg : (const T*)nullptr, ldg, sink, bias, bias_len, ldo, status);
+                gate ? (const T*)gate + (size_t)t0 * ldg : (const T*)nullptr, ldg, sink, bias, bias_len, ldo, keep_first, status);
         });
     }
     return qi::check_launch("attention_generic");
@@ -190,7 +194,7 @@ extern "C" int qi_attention_generic_sink(const void* q, void* out, int dtype, co
                                        long long ldg, const float* sink, int* status, cudaStream_t stream) {
     return qi_attention_generic_bias(q, out, dtype, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, positions,
                                      token_req, n_tokens, nq, nkv, d, dv, scale, softcap, out_scale, window, chunk, gate, ldg,
-                                     sink, nullptr, 0, (long long)nq * dv, status, stream);
+                                     sink, nullptr, 0, (long long)nq * dv, 0, status, stream);
 }
 
 extern "C" int qi_attention_generic_cap(const void* q, void* out, int dtype, const void* k_pages,

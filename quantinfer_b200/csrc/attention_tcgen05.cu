@@ -264,7 +264,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                                       float scale_log2e, int window, int* __restrict__ status, int n_ranges,
                                       float* __restrict__ ws_o, float* __restrict__ ws_ml, int chunk,
                                       const qi::bf16* __restrict__ gate, long long ldg, float cap, float cap_pre,
-                                      float out_scale, const float* __restrict__ sink, const float* __restrict__ bias, int bias_len, long long ldo) {
+                                      float out_scale, const float* __restrict__ sink, const float* __restrict__ bias, int bias_len, long long ldo, int keep_first) {
     extern __shared__ uint8_t smem_raw[];
     using B = Bars;
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -297,13 +297,18 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
     // With n_ranges > 1 the key tiles of these query rows are cut into that many ranges, one CTA each
     // (blockIdx.z); every CTA leaves its rows' reference, sum and accumulator in the workspace and a
     // second kernel merges them. A long context then gives enough CTAs to fill the GPU's last round.
+    // Kept first keys: the tiles that hold them and lie wholly before the others come first, `head` of them from
+    // position 0 (of this CTA's own tiles, j < head).
     int t_begin = (lo / BN) * BN;
-    int n_tiles = (hi - t_begin + BN - 1) / BN;
+    int head = min((keep_first + BN - 1) / BN, t_begin / BN), head0 = 0;
+    int n_tiles = head + (hi - t_begin + BN - 1) / BN;
     if (n_ranges > 1) {
         const int per = (n_tiles + n_ranges - 1) / n_ranges;
         const int first = (int)blockIdx.z * per;
         const int count = max(min(n_tiles - first, per), 0);
-        t_begin += first * BN;
+        t_begin += max(first - head, 0) * BN;
+        head0 = min(first, head) * BN;
+        head = min(max(head - first, 0), count);
         n_tiles = count;
         if (count == 0) {    // nothing of the rows' keys falls into this range: an empty partial
             const int row = threadIdx.x;
@@ -319,7 +324,8 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
         }
     }
     const int blk0 = t_begin / page_size;
-    const int n_blk = min(min((t_begin + n_tiles * BN + page_size - 1) / page_size, max_blocks) - blk0, kMaxTableEntries);
+    const int n_blk = min(min((t_begin + (n_tiles - head) * BN + page_size - 1) / page_size, max_blocks) - blk0, kMaxTableEntries);
+    auto tile_start = [&](int j) { return j < head ? head0 + j * BN : t_begin + (j - head) * BN; };
     for (int i = threadIdx.x; i < n_blk; i += blockDim.x) s_table[i] = table[blk0 + i];
 
     if (threadIdx.x == 0) {
@@ -375,13 +381,14 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                 const uint32_t dst = kv_s + s * 2 * kKVBytes + (is_v ? kKVBytes : 0);
                 const CUtensorMap* map = is_v ? &map_v : &map_k;
                 mbar_expect_tx(full, kKVBytes);
-                const int t0 = t_begin + j * BN;
+                const int t0 = tile_start(j);
                 for (int r0 = 0; r0 < BN; r0 += box_rows) {
                     const int key = t0 + r0;
                     const int blk = key / page_size - blk0;
-                    int page = blk < n_blk ? s_table[blk] : -1;
+                    // (kept keys before the window: their pages are looked up in the table itself)
+                    int page = j < head ? (key < keep_first ? table[key / page_size] : -1) : blk < n_blk ? s_table[blk] : -1;
                     if (page < 0 || page >= num_pages) {
-                        if (!is_v && key < hi && key + box_rows > lo && status) atomicOr(status, qi::kStatusBadPage);
+                        if (!is_v && key < hi && (key + box_rows > lo || key < keep_first) && status) atomicOr(status, qi::kStatusBadPage);
                         page = 0;
                     }
                     const int row = (page * nkv + hk) * page_size + (key % page_size);
@@ -467,11 +474,17 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
         bool ok = true;
         for (int j = 0; j < n_tiles && ok; ++j) {
             const uint32_t u = (uint32_t)j;
-            const int t0 = t_begin + j * BN;
+            const int t0 = tile_start(j);
             if (!mbar_wait(bars + B::s_full, u & 1u, abort_flag)) { ok = false; break; }
             tc_fence_after();
             int c_hi = min(min(pos, hi - 1) - t0 + 1, BN);
             int c_lo = max(max(lo, window > 0 ? pos - window + 1 : 0), chunk > 0 ? pos / chunk * chunk : 0) - t0;
+            const int kept = keep_first - t0;       // columns 0 .. kept - 1 hold kept keys
+            int gap_lo = BN, gap_hi = 0;            // columns between the kept keys and the row's own first one
+            if (kept > 0) {
+                if (c_lo > kept) { gap_lo = kept; gap_hi = c_lo; }
+                c_lo = 0;
+            }
             if (c_lo < 0) c_lo = 0;
             if (c_hi < 0) c_hi = 0;
             uint32_t sv[BN];
@@ -506,6 +519,11 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, cons
                         sv[c] = __float_as_uint(fmaf(b, 1.4426950408889634f, __uint_as_float(sv[c]) * scale_log2e));
                     }
                 }
+            }
+            if (__any_sync(0xffffffffu, gap_lo < gap_hi)) {        // only tiles that hold kept keys
+#pragma unroll
+                for (int c = 0; c < BN; ++c)
+                    if (c >= gap_lo && c < gap_hi) sv[c] = 0xff800000u;
             }
             // a tile that lies wholly inside every row's span takes the code without the comparisons
             const bool interior = __all_sync(0xffffffffu, c_lo == 0 && c_hi == BN);
@@ -690,6 +708,7 @@ extern "C" int qi_attention_prefill_tcgen05_supported(int nq, int nkv, int d, in
 // applied) becomes c tanh(s / c) before the softmax. out_scale multiplies the result. sink (or null): float32 [nq]; the
 // softmax's denominator of head h holds exp(sink[h]) once more. bias (or null): float32 [nq, bias_len]; a key n positions
 // back adds bias[h, min(n, bias_len - 1)] to its score (after the cap). ldo: elements from one row of out to the next.
+// keep_first: keys 0 .. keep_first - 1 stay visible behind a window or chunk.
 extern "C" int qi_attention_prefill_tcgen05_bias(const void* q, void* out, const void* k_pages, const void* v_pages,
                                                const int* block_table, int max_blocks, int page_size, int num_pages,
                                                const int* q_start, const int* start_pos, const int* tile_req,
@@ -697,7 +716,8 @@ extern "C" int qi_attention_prefill_tcgen05_bias(const void* q, void* out, const
                                                float scale, int window, int chunk, const void* gate, long long ldg,
                                                int n_ranges, float* workspace, int* status, float softcap, float out_scale,
                                                const float* sink, const float* bias, int bias_len, long long ldo,
-                                               cudaStream_t stream) {
+                                               int keep_first, cudaStream_t stream) {
+    QI_REQUIRE(keep_first >= 0, "attention_prefill_tcgen05: keep_first must be >= 0 (0 = none)");
     QI_REQUIRE(ldo >= (long long)nq * D && ldo % 8 == 0 && ((uintptr_t)out & 15) == 0,
                "attention_prefill_tcgen05: the output must be 16-byte aligned with rows a multiple of 8 elements apart");
     QI_REQUIRE(!bias || bias_len > 0, "attention_prefill_tcgen05: an empty distance bias");
@@ -734,7 +754,7 @@ extern "C" int qi_attention_prefill_tcgen05_bias(const void* q, void* out, const
     qi::launch(attention_prefill_tcgen05_kernel, dim3(nq, n_tiles, n_ranges), dim3(kThreads), kSmemBytes, stream, mq, mk, mv,
                (qi::bf16*)out, block_table, max_blocks, page_size, box_rows, num_pages, q_start, start_pos, tile_req,
                tile_q0, nq, nkv, softcap > 0.f ? log2e : scale * log2e, window, status, n_ranges, ws_o, ws_ml, chunk,
-               (const qi::bf16*)gate, ldg, softcap, cap_pre, out_scale, sink, bias, bias_len, ldo);
+               (const qi::bf16*)gate, ldg, softcap, cap_pre, out_scale, sink, bias, bias_len, ldo, keep_first);
     if (n_ranges > 1) {
         if (int rc = qi::check_launch("attention_prefill_tcgen05")) return rc;
         qi::launch(attention_prefill_merge_kernel, dim3(nq, n_tokens), dim3(128), 0, stream, (const float*)ws_o,
@@ -753,7 +773,7 @@ extern "C" int qi_attention_prefill_tcgen05_ex(const void* q, void* out, const v
                                                cudaStream_t stream) {
     return qi_attention_prefill_tcgen05_bias(q, out, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, q_start,
                                              start_pos, tile_req, tile_q0, n_tiles, n_tokens, nq, nkv, d, scale, window, chunk,
-                                             gate, ldg, n_ranges, workspace, status, softcap, out_scale, nullptr, nullptr, 0, (long long)nq * D, stream);
+                                             gate, ldg, n_ranges, workspace, status, softcap, out_scale, nullptr, nullptr, 0, (long long)nq * D, 0, stream);
 }
 
 extern "C" int qi_attention_prefill_tcgen05(const void* q, void* out, const void* k_pages, const void* v_pages,

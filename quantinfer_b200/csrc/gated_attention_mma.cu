@@ -6,13 +6,14 @@
 //     s_ij = cap((q_i . k_j) * scale)    for lo(i) <= j <= i,   lo(i) = max(start of i's chunk, i - window + 1, 0)
 //     out_i = (sum_j softmax(s_i)_j v_j) * sigmoid(gate_i) * out_scale      cap(s) = c tanh(s / c), or s without a cap
 //
-// A distance bias (optional) adds to s_ij a number per head that depends on i - j alone (after the cap).
+// A distance bias (optional) adds to s_ij a number per head that depends on i - j alone (after the cap). The sequence's first
+// `keep_first` keys (optional) stay visible whatever the bounds say: j < keep_first beside lo(i) <= j.
 //
 // One kernel serves prompts, portions and single decode tokens: a CTA of four warps takes up to 64
 // consecutive query rows of ONE step entry and one query head (the tiles are found on the device from
 // q_start, so the launch can sit in a CUDA graph), walks the keys its rows can see in tiles of 64 that
 // start at multiples of 64 of the ABSOLUTE position (so a row's sums do not depend on where a prompt
-// was cut), with the softmax evaluated online; the next tile is requested with cp.async into a second buffer
+// was cut; first the tiles that hold kept keys and lie wholly before the others), with the softmax evaluated online; the next tile is requested with cp.async into a second buffer
 // while the current one is multiplied. Keys before the first visible one are zero-filled and
 // never looked up: their pages may have gone back to the pool. Head sizes are padded with zeros to the
 // next of 32, 64, 96, 128 in shared memory.
@@ -23,6 +24,18 @@
 namespace {
 
 constexpr int kQT = 64, kKT = 64, kThreads = 128, kPad = 8;
+
+// The key tiles of a query tile whose first visible key (without the kept ones) is `lo` and whose last is `hi`: `head`
+// tiles from position 0 for the kept keys before that, then the tiles from `first` to the one that holds `hi`.
+struct KeyTiles {
+    int head, first, count;
+    __device__ KeyTiles(int lo, int hi, int keep_first) {
+        first = lo / kKT * kKT;
+        head = min((keep_first + kKT - 1) / kKT, first / kKT);
+        count = head + (hi - first) / kKT + 1;
+    }
+    __device__ int start(int it) const { return it < head ? it * kKT : first + (it - head) * kKT; }
+};
 
 __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -75,7 +88,8 @@ gated_attention_mma_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restrict_
                            int page_size, int num_pages, const int* __restrict__ q_start, const int* __restrict__ start_pos,
                            int n_entries, int nq, int nkv, int d, int dv, float scale_log2e, float softcap, float out_scale,
                            int window, int chunk, const qi::bf16* __restrict__ gate, long long ldg, const float* __restrict__ sink,
-                           const float* __restrict__ bias, int bias_len, int n_ranges, float* __restrict__ ws_o, float* __restrict__ ws_ml, long long ldo, int* __restrict__ status) {
+                           const float* __restrict__ bias, int bias_len, int n_ranges, float* __restrict__ ws_o, float* __restrict__ ws_ml, long long ldo,
+                           int keep_first, int* __restrict__ status) {
     extern __shared__ __align__(16) uint8_t smem_raw[];
     constexpr int SK = DK + kPad, SV = DV + kPad;
     qi::bf16* Qs = reinterpret_cast<qi::bf16*>(smem_raw);       // [kQT][SK]
@@ -139,7 +153,7 @@ gated_attention_mma_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restrict_
     auto request_tile = [&](int t0, int buf) {
         auto page_row = [&](int r, const qi::bf16* pages, int width) -> const qi::bf16* {
             const int key = t0 + r;
-            if (key < lo_min || key > hi) return nullptr;
+            if ((key < lo_min && key >= keep_first) || key > hi) return nullptr;
             const int page = table[key / page_size];
             if (page < 0 || page >= num_pages) { bad_page = true; return nullptr; }
             return pages + (((size_t)page * nkv + hk) * page_size + (key % page_size)) * (size_t)width;
@@ -148,18 +162,20 @@ gated_attention_mma_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restrict_
         fill_tile_async(Vbuf + (size_t)buf * kKT * SV, SV, kKT, dv, DV, k_pages, [&](int r) { return page_row(r, v_pages, dv); });
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    int t_first = lo_min / kKT * kKT, t_last = hi;
+    const KeyTiles tiles(lo_min, hi, keep_first);
+    int it0 = 0, it1 = tiles.count;
     if (n_ranges > 1) {
         // the tile's key tiles in n_ranges equal parts, one a CTA along grid.z; a merge kernel adds the parts
-        const int per = ((hi - t_first) / kKT + n_ranges) / n_ranges;
-        t_first += (int)blockIdx.z * per * kKT;
-        t_last = min(hi, t_first + per * kKT - 1);
+        const int per = (tiles.count + n_ranges - 1) / n_ranges;
+        it0 = (int)blockIdx.z * per;
+        it1 = min(it1, it0 + per);
     }
     int buf = 0;
-    if (t_first <= t_last) request_tile(t_first, 0);
-    for (int t0 = t_first; t0 <= t_last; t0 += kKT, buf ^= 1) {
-        if (t0 + kKT <= t_last) {        // the next tile lands while this one is multiplied
-            request_tile(t0 + kKT, buf ^ 1);
+    if (it0 < it1) request_tile(tiles.start(it0), 0);
+    for (int it = it0; it < it1; ++it, buf ^= 1) {
+        const int t0 = tiles.start(it);
+        if (it + 1 < it1) {        // the next tile lands while this one is multiplied
+            request_tile(tiles.start(it + 1), buf ^ 1);
             asm volatile("cp.async.wait_group 1;" ::: "memory");
         } else {
             asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -215,8 +231,8 @@ gated_attention_mma_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restrict_
 #pragma unroll
             for (int j = 0; j < 2; ++j) {
                 const int key = t0 + n * 8 + (lane & 3) * 2 + j;
-                s[n][j] = (key >= loA && key <= pA && rA < rows) ? fmaf(s[n][j], mul, add) : -INFINITY;
-                s[n][2 + j] = (key >= loB && key <= pB && rB < rows) ? fmaf(s[n][2 + j], mul, add) : -INFINITY;
+                s[n][j] = ((key >= loA || key < keep_first) && key <= pA && rA < rows) ? fmaf(s[n][j], mul, add) : -INFINITY;
+                s[n][2 + j] = ((key >= loB || key < keep_first) && key <= pB && rB < rows) ? fmaf(s[n][2 + j], mul, add) : -INFINITY;
                 tmA = fmaxf(tmA, s[n][j]);
                 tmB = fmaxf(tmB, s[n][2 + j]);
             }
@@ -325,7 +341,7 @@ gated_attention_decode_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restri
                               int nq, int nkv, int d, int dv, float scale_log2e, float softcap, float out_scale,
                               int window, int chunk, const qi::bf16* __restrict__ gate, long long ldg, const float* __restrict__ sink,
                               const float* __restrict__ bias, int bias_len, int n_ranges, float* __restrict__ ws_o,
-                              float* __restrict__ ws_ml, long long ldo, int* __restrict__ status) {
+                              float* __restrict__ ws_ml, long long ldo, int keep_first, int* __restrict__ status) {
     extern __shared__ __align__(16) uint8_t smem_raw[];
     constexpr int SK = DK + kPad, SV = DV + kPad;
     qi::bf16* Qs = reinterpret_cast<qi::bf16*>(smem_raw);       // [kGroupRows][SK]
@@ -345,7 +361,7 @@ gated_attention_decode_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restri
     auto request_tile = [&](int t0, int buf) {
         auto page_row = [&](int r, const qi::bf16* pages, int width) -> const qi::bf16* {
             const int key = t0 + r;
-            if (key < lo || key > pos) return nullptr;
+            if ((key < lo && key >= keep_first) || key > pos) return nullptr;
             const int page = table[key / page_size];
             if (page < 0 || page >= num_pages) { bad_page = true; return nullptr; }
             return pages + (((size_t)page * nkv + hk) * page_size + (key % page_size)) * (size_t)width;
@@ -354,14 +370,15 @@ gated_attention_decode_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restri
         fill_tile_async(Vbuf + (size_t)buf * kKT * SV, SV, kKT, dv, DV, k_pages, [&](int r) { return page_row(r, v_pages, dv); });
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    int t_first = lo / kKT * kKT, t_last = pos;
+    const KeyTiles tiles(lo, pos, keep_first);
+    int it0 = 0, it1 = tiles.count;
     if (n_ranges > 1) {
-        const int per = ((pos - t_first) / kKT + n_ranges) / n_ranges;
-        t_first += (int)blockIdx.z * per * kKT;
-        t_last = min(pos, t_first + per * kKT - 1);
+        const int per = (tiles.count + n_ranges - 1) / n_ranges;
+        it0 = (int)blockIdx.z * per;
+        it1 = min(it1, it0 + per);
     }
     int buf = 0;
-    if (t_first <= t_last) request_tile(t_first, 0);
+    if (it0 < it1) request_tile(tiles.start(it0), 0);
     fill_tile(Qs, SK, kGroupRows, d, DK, [&](int r) -> const qi::bf16* {
         return r < group ? q + ((size_t)t * nq + h0 + r) * d : nullptr;
     });
@@ -386,9 +403,10 @@ gated_attention_decode_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restri
 #pragma unroll
     for (int n = 0; n < DV / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
 
-    for (int t0 = t_first; t0 <= t_last; t0 += kKT, buf ^= 1) {
-        if (t0 + kKT <= t_last) {        // the next tile lands while this one is multiplied
-            request_tile(t0 + kKT, buf ^ 1);
+    for (int it = it0; it < it1; ++it, buf ^= 1) {
+        const int t0 = tiles.start(it);
+        if (it + 1 < it1) {        // the next tile lands while this one is multiplied
+            request_tile(tiles.start(it + 1), buf ^ 1);
             asm volatile("cp.async.wait_group 1;" ::: "memory");
         } else {
             asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -418,7 +436,7 @@ gated_attention_decode_kernel(const qi::bf16* __restrict__ q, qi::bf16* __restri
                     a = c * tanhf(a / c);
                     b = c * tanhf(b / c);
                 }
-                const bool visible = key >= lo && key <= pos;
+                const bool visible = (key >= lo || key < keep_first) && key <= pos;
                 if (bias) {
                     const int back = min(max(pos - key, 0), bias_len - 1);
                     a = fmaf(__ldg(biasA + back), kLog2e, a);
@@ -538,7 +556,7 @@ template <int DK, int DV>
 int launch_one(dim3 grid, cudaStream_t stream, const void* q, void* out, const void* k_pages, const void* v_pages,
                const int* block_table, int max_blocks, int page_size, int num_pages, const int* q_start, const int* start_pos,
                int n_entries, int nq, int nkv, int d, int dv, float scale_log2e, float softcap, float out_scale, int window, int chunk,
-               const void* gate, long long ldg, const float* sink, const float* bias, int bias_len, int n_ranges, float* ws_o, float* ws_ml, int n_tokens, int grouped, long long ldo, int* status) {
+               const void* gate, long long ldg, const float* sink, const float* bias, int bias_len, int n_ranges, float* ws_o, float* ws_ml, int n_tokens, int grouped, long long ldo, int keep_first, int* status) {
     const size_t smem = sizeof(qi::bf16) * ((size_t)((grouped ? kGroupRows : kQT) + 2 * kKT) * (DK + kPad) + (size_t)2 * kKT * (DV + kPad));
     static bool raised[2] = {false, false};
     if (!raised[grouped] && smem > 48 * 1024) {
@@ -550,12 +568,12 @@ int launch_one(dim3 grid, cudaStream_t stream, const void* q, void* out, const v
         qi::launch(gated_attention_decode_kernel<DK, DV>, grid, dim3(kThreads), smem, stream, (const qi::bf16*)q, (qi::bf16*)out,
                    (const qi::bf16*)k_pages, (const qi::bf16*)v_pages, block_table, max_blocks, page_size, num_pages, q_start, start_pos,
                    nq, nkv, d, dv, scale_log2e, softcap, out_scale, window, chunk, (const qi::bf16*)gate, ldg, sink, bias, bias_len, n_ranges,
-                   ws_o, ws_ml, ldo, status);
+                   ws_o, ws_ml, ldo, keep_first, status);
     else
         qi::launch(gated_attention_mma_kernel<DK, DV>, grid, dim3(kThreads), smem, stream, (const qi::bf16*)q, (qi::bf16*)out,
                    (const qi::bf16*)k_pages, (const qi::bf16*)v_pages, block_table, max_blocks, page_size, num_pages, q_start, start_pos,
                    n_entries, nq, nkv, d, dv, scale_log2e, softcap, out_scale, window, chunk, (const qi::bf16*)gate, ldg, sink, bias, bias_len,
-                   n_ranges, ws_o, ws_ml, ldo, status);
+                   n_ranges, ws_o, ws_ml, ldo, keep_first, status);
     if (n_ranges > 1) {
         if (int rc = qi::check_launch("gated_attention_mma")) return rc;
         qi::launch(gated_attention_merge_kernel, dim3(nq, n_tokens), dim3(128), 0, stream, (const float*)ws_o, (const float*)ws_ml,
@@ -577,7 +595,7 @@ extern "C" int qi_gated_attention_mma_supported(int nq, int nkv, int d, int dv) 
 // float32 [nq]; the softmax's denominator of head h holds exp(sink[h]) once more.
 // bias (may be null): float32 [nq, bias_len]; a key n positions back adds bias[h, min(n, bias_len - 1)] to its score.
 // grouped: every entry has one token, and the query heads of a key head (up to 16) are the rows of one tile. ldo: elements from
-// one row of out to the next (even).
+// one row of out to the next (even). keep_first: keys 0 .. keep_first - 1 stay visible behind a window or chunk.
 // n_ranges > 1 (steps of single tokens over long contexts): every query tile's keys are cut into that many ranges over
 // separate CTAs and a second kernel adds the parts; `workspace` must then hold n_tokens * nq * n_ranges * (dv + 2) floats.
 extern "C" int qi_gated_attention_mma_bias(const void* q, void* out, const void* k_pages, const void* v_pages, const int* block_table,
@@ -585,7 +603,8 @@ extern "C" int qi_gated_attention_mma_bias(const void* q, void* out, const void*
                                       int n_entries, int n_tokens, int nq, int nkv, int d, int dv, float scale, float softcap,
                                       float out_scale, int window, int chunk, const void* gate, long long ldg, const float* sink,
                                       const float* bias, int bias_len, int n_ranges, float* workspace, int grouped, long long ldo,
-                                      int* status, cudaStream_t stream) {
+                                      int keep_first, int* status, cudaStream_t stream) {
+    QI_REQUIRE(keep_first >= 0, "gated_attention_mma: keep_first must be >= 0 (0 = none)");
     QI_REQUIRE(ldo >= (long long)nq * dv && ldo % 2 == 0 && ((uintptr_t)out & 3) == 0, "gated_attention_mma: the output's rows are too short or odd");
     QI_REQUIRE(!grouped || (n_tokens == n_entries && nkv > 0 && nq / nkv <= kGroupRows && nkv <= 65535),
                "gated_attention_mma: the grouped form takes steps of single tokens and up to %d query heads a key head", kGroupRows);
@@ -605,7 +624,7 @@ extern "C" int qi_gated_attention_mma_bias(const void* q, void* out, const void*
     const float sl = scale * 1.4426950408889634f;
 #define QI_GA(DKP, DVP)                                                                                                      \
     return launch_one<DKP, DVP>(grid, stream, q, out, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, q_start, \
-                                start_pos, n_entries, nq, nkv, d, dv, sl, softcap, out_scale, window, chunk, gate, ldg, sink, bias, bias_len, n_ranges, ws_o, ws_ml, n_tokens, grouped, ldo, status)
+                                start_pos, n_entries, nq, nkv, d, dv, sl, softcap, out_scale, window, chunk, gate, ldg, sink, bias, bias_len, n_ranges, ws_o, ws_ml, n_tokens, grouped, ldo, keep_first, status)
 #define QI_GA_ROW(DKP)                                   \
     switch (padded(dv)) {                                \
         case 32: QI_GA(DKP, 32);                         \
@@ -646,5 +665,5 @@ extern "C" int qi_gated_attention_mma_sink(const void* q, void* out, const void*
                                       int* status, cudaStream_t stream) {
     return qi_gated_attention_mma_bias(q, out, k_pages, v_pages, block_table, max_blocks, page_size, num_pages, q_start, start_pos,
                                          n_entries, n_tokens, nq, nkv, d, dv, scale, softcap, out_scale, window, chunk, gate, ldg, sink, nullptr, 0, 1,
-                                         nullptr, 0, (long long)nq * dv, status, stream);
+                                         nullptr, 0, (long long)nq * dv, 0, status, stream);
 }

@@ -21,6 +21,11 @@
 // `half_split`, (i, i + rot_dims / 2), turns by the angle position * inv_freq[i], computed here in 32-bit (no
 // table, so no limit on positions); cos and sin are multiplied by `magnitude` (1 for the plain rotation).
 //
+// qi_latent_down: for queries that come through a latent of their own. Per token, from the row of the fused projection [query
+// latent | latent | rotated key part], whole or as the partial sums of a product whose contraction was cut: normalises the
+// query latent (its own gain) for the product that makes the heads' queries, and normalises, rotates and caches the rest as
+// qi_latent_prepare does.
+//
 // qi_latent_attention_generic: 32-bit arithmetic for any sizes; one block per (token, head).
 #include "common.cuh"
 
@@ -95,6 +100,60 @@ latent_prepare_kernel(const TP* __restrict__ proj, long long ldp, int kv_off, T*
             v = second ? b * cs[i] + a * sn[i] : a * cs[i] - b * sn[i];
         } else {
             v = qi::to_f32<TP>(z[R + j]);
+        }
+        dst[R + j] = qi::from_f32<T>(v);
+    }
+}
+
+template <typename TP, typename T>
+__global__ void __launch_bounds__(128)
+latent_down_kernel(const TP* __restrict__ proj, int parts, size_t part_stride, long long ldp, int Q, const float* __restrict__ q_gain,
+                   T* __restrict__ cq, const float* __restrict__ gain, float eps, const float* __restrict__ inv_freq, int rot_dims,
+                   const int* __restrict__ positions, const int* __restrict__ token_req, const int* __restrict__ block_table,
+                   int max_blocks, int page_size, int num_pages, T* __restrict__ cache, int r, int R, int half_split, float magnitude,
+                   int* __restrict__ status) {
+    extern __shared__ float smem[];
+    float* row = smem;                    // [Q + R + r]: the projected row, parts added
+    __shared__ float scratch[32];
+    qi::pdl_wait();
+    const int t = blockIdx.x, total = Q + R + r;
+    const TP* src = proj + (size_t)t * ldp;
+    float sq = 0.f, sc = 0.f;
+    for (int i = threadIdx.x; i < total; i += blockDim.x) {
+        float v = qi::to_f32<TP>(src[i]);
+#pragma unroll 4
+        for (int k = 1; k < parts; ++k) v += qi::to_f32<TP>(src[k * part_stride + i]);
+        row[i] = v;
+        if (i < Q) sq = fmaf(v, v, sq);
+        else if (i < Q + R) sc = fmaf(v, v, sc);
+    }
+    const float q_inv = 1.0f / sqrtf(qi::block_sum(sq, scratch) / (float)Q + eps);
+    const float c_inv = 1.0f / sqrtf(qi::block_sum(sc, scratch) / (float)R + eps);
+    __syncthreads();
+    for (int i = threadIdx.x; i < Q; i += blockDim.x) cq[(size_t)t * Q + i] = qi::from_f32<T>(row[i] * q_inv * q_gain[i]);
+    const int pos = positions[t];
+    if (pos < 0) {
+        if (threadIdx.x == 0 && status) atomicOr(status, qi::kStatusBadRange);
+        return;
+    }
+    const int page = block_table[(size_t)token_req[t] * max_blocks + pos / page_size];
+    if (page < 0 || page >= num_pages) {
+        if (threadIdx.x == 0 && status) atomicOr(status, qi::kStatusBadPage);
+        return;
+    }
+    T* dst = cache + ((size_t)page * page_size + pos % page_size) * (R + r);
+    const float* z = row + Q;
+    for (int i = threadIdx.x; i < R; i += blockDim.x) dst[i] = qi::from_f32<T>(z[i] * c_inv * gain[i]);
+    const int half = rot_dims >> 1;
+    for (int j = threadIdx.x; j < r; j += blockDim.x) {
+        float v = z[R + j];
+        if (j < rot_dims) {
+            const int i = half_split ? (j < half ? j : j - half) : j >> 1;
+            const bool second = half_split ? j >= half : (j & 1);
+            const float a = z[R + (half_split ? i : 2 * i)], b = z[R + (half_split ? i + half : 2 * i + 1)];
+            float sn, cs;
+            sincosf((float)pos * inv_freq[i], &sn, &cs);
+            v = (second ? b * cs + a * sn : a * cs - b * sn) * magnitude;
         }
         dst[R + j] = qi::from_f32<T>(v);
     }
@@ -229,6 +288,31 @@ extern "C" int qi_latent_prepare(const void* proj, int proj_dtype, long long ldp
         });
     });
     return qi::check_launch("latent_prepare");
+}
+
+// proj [parts, n, ldp] in `proj_dtype` (parts part_stride elements apart, added in their order): columns 0 .. Q - 1 the query
+// latent, then R + r of the latent projection. cq [n, Q] in `dtype`; cache [num_pages, page_size, R + r] in `dtype`; q_gain float32
+// [Q], gain float32 [R]; inv_freq float32 [rot_dims / 2].
+extern "C" int qi_latent_down(const void* proj, int proj_dtype, int parts, long long part_stride, long long ldp, int Q,
+                              const float* q_gain, void* cq, int dtype, const float* gain, float eps, const float* inv_freq,
+                              int rot_dims, const int* positions, const int* token_req, const int* block_table, int max_blocks,
+                              int page_size, int num_pages, void* cache, int n_tokens, int r, int R, int half_split,
+                              float magnitude, int* status, cudaStream_t stream) {
+    QI_REQUIRE(n_tokens >= 0 && Q > 0 && r >= 0 && R > 0 && eps > 0.f, "latent_down: bad sizes or eps");
+    QI_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= r && (rot_dims == 0 || inv_freq), "latent_down: %d rotated coordinates do not fit a part of %d, or their frequencies are missing", rot_dims, r);
+    QI_REQUIRE(parts >= 1 && ldp >= (long long)Q + R + r && (parts == 1 || part_stride >= (long long)n_tokens * ldp), "latent_down: the projection's rows are too short");
+    QI_REQUIRE(cache && gain && q_gain && cq && block_table && page_size > 0 && max_blocks > 0 && num_pages > 0, "latent_down: the cache or a gain is missing");
+    const size_t smem = sizeof(float) * (size_t)(Q + R + r);
+    QI_REQUIRE(smem <= 47 * 1024, "latent_down: a row of %d + %d + %d is too wide for this kernel", Q, R, r);
+    if (n_tokens == 0) return 0;
+    QI_DISPATCH_DTYPE(proj_dtype, TP, {
+        QI_DISPATCH_DTYPE(dtype, T, {
+            qi::launch(latent_down_kernel<TP, T>, dim3(n_tokens), dim3(128), smem, stream, (const TP*)proj, parts, (size_t)part_stride, ldp,
+                       Q, q_gain, (T*)cq, gain, eps, inv_freq, rot_dims, positions, token_req, block_table, max_blocks, page_size,
+                       num_pages, (T*)cache, r, R, half_split, magnitude, status);
+        });
+    });
+    return qi::check_launch("latent_down");
 }
 
 // q [n, H, W], out [n, H, R], cache [num_pages, page_size, W], all in `dtype`; sink float32 [H] or null.

@@ -1,18 +1,22 @@
 // Mixture of experts: routing, grouping of the tokens by expert, the experts' products as one grouped
 // launch, and the weighted sum.
 //
-//   moe_route     per token: s = softmax(router logits) over all experts (32-bit); the `top` experts with the
-//                 largest s + correction are chosen (ties: the lower index); their weights are their s divided
-//                 by the sum of the chosen s (+ 1e-20) and multiplied by `scale`.
+//   moe_route     per token: s = softmax(router logits) over all experts, or sigmoid(router logits) (32-bit); the
+//                 `top` experts with the largest s + correction are chosen (ties: the lower index); their weights
+//                 are their s divided by the sum of the chosen s (+ 1e-20), or s as they are, times `scale`.
 //   moe_group     the (token, choice) pairs sorted by expert: offsets per expert, the pairs' order, each pair's
 //                 place in that order, and a list of row tiles (expert, first row, rows) of at most `tile` rows
 //                 that no expert shares with another. One block; everything stays on the device, so a step
 //                 never waits for the host to learn how many tokens an expert got.
 //   moe_gemm      y[i] = W[expert of row i] . x[source of row i] over the sorted rows i, 32-bit products and
 //                 sums with k ascending (the 32-bit path, and any type the tensor-core kernel does not take);
-//                 a row's result does not depend on which other rows its expert got.
-//   moe_combine   out[t] = sum_k weight[t, k] * y[place of (t, k)] (+ shared[t]), k ascending, 32-bit.
+//                 a row's result does not depend on which other rows its expert got. Optional epilogue for a W
+//                 whose rows are (gate, up) pairs: silu(w g) w u, w the pair's weight, for designs whose weight
+//                 multiplies an expert's input (the products are linear in it).
+//   moe_combine   out[t] = sum_k weight[t, k] * y[place of (t, k)] (+ shared[t]) (+ another branch's output, which
+//                 may still be partial sums), k ascending, 32-bit; without weights the plain sum.
 #include "common.cuh"
+#include "vec8.cuh"
 
 #include <math.h>
 
@@ -22,7 +26,7 @@ constexpr int kMaxPerLane = 32;   // experts a lane holds: up to 1,024 experts
 
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int* __restrict__ ids,
-                 float* __restrict__ weights, int n, int E, int top, float scale) {
+                 float* __restrict__ weights, int n, int E, int top, float scale, int sigmoid, int normalize) {
     qi::pdl_wait();
     const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (t >= n) return;
@@ -47,7 +51,7 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ cor
 #pragma unroll
     for (int i = 0; i < kMaxPerLane; ++i) {
         const int e = lane + 32 * i;
-        s[i] = s[i] / sum;
+        s[i] = sigmoid ? (e < E ? 1.0f / (1.0f + expf(-z[e])) : 0.f) : s[i] / sum;
         c[i] = e < E ? s[i] + (correction ? correction[e] : 0.f) : -INFINITY;
     }
     float chosen_sum = 0.f;
@@ -77,7 +81,7 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ cor
             weights[(size_t)t * top + k] = sc;
         }
     }
-    const float inv = scale / (chosen_sum + 1e-20f);
+    const float inv = normalize ? scale / (chosen_sum + 1e-20f) : scale;
     for (int k = lane; k < top; k += 32) weights[(size_t)t * top + k] *= inv;
 }
 
@@ -130,13 +134,19 @@ moe_group_kernel(const int* __restrict__ ids, int n_pairs, int E, int tile, int 
 
 constexpr int BM = 32, BN = 64, BK = 16, TM = 2, TN = 4;
 
+// silu(w g) * (w u)
+__device__ __forceinline__ float scaled_silu_mul(float g, float u, float w) {
+    g *= w;
+    return g / (1.0f + expf(-g)) * (u * w);
+}
+
 // Rows are the sorted (token, choice) pairs; a tile's rows belong to one expert. Source row of sorted row i:
 // order[i] / top when `gather` (the experts read the tokens' rows), else i (they read rows already in sorted order).
 template <typename TX, typename TW, typename TY>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TY* __restrict__ y, const int* __restrict__ tiles,
                 const int* __restrict__ order, int top, int gather, int N, int K, long long ldx, long long ldy, int n_src,
-                int n_rows, int n_experts) {
+                int n_rows, int n_experts, int epilogue, const float* __restrict__ pair_scale) {
     __shared__ float xs[BK][BM + 4];
     __shared__ float ws[BK][BN + 4];
     __shared__ int src_row[BM];
@@ -190,6 +200,15 @@ moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TY* __restri
     for (int i = 0; i < TM; ++i) {
         const int m = ty * TM + i;
         if (m >= rows) continue;
+        if (epilogue) {
+            const float w = pair_scale ? pair_scale[order[row0 + m]] : 1.f;
+#pragma unroll
+            for (int j = 0; j < TN; j += 2) {
+                const int n = n0 + tx * TN + j;
+                if (n + 1 < N) y[(size_t)(row0 + m) * ldy + (n >> 1)] = qi::from_f32<TY>(scaled_silu_mul(acc[i][j], acc[i][j + 1], w));
+            }
+            continue;
+        }
 #pragma unroll
         for (int j = 0; j < TN; ++j) {
             const int n = n0 + tx * TN + j;
@@ -211,7 +230,8 @@ __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], uint32_t a0, uint3
 __global__ void __launch_bounds__(128)
 moe_gemm_mma_kernel(const qi::bf16* __restrict__ x, const qi::bf16* __restrict__ w, qi::bf16* __restrict__ y,
                     const int* __restrict__ tiles, const int* __restrict__ order, int top, int gather, int N, int K,
-                    long long ldx, long long ldy, int n_src, int n_rows, int n_experts) {
+                    long long ldx, long long ldy, int n_src, int n_rows, int n_experts, int epilogue,
+                    const float* __restrict__ pair_scale) {
     __shared__ __align__(16) qi::bf16 As[BM][MK + MPAD];
     __shared__ __align__(16) qi::bf16 Bs[MN][MK + MPAD];
     __shared__ int src_row[BM];
@@ -285,6 +305,12 @@ moe_gemm_mma_kernel(const qi::bf16* __restrict__ x, const qi::bf16* __restrict__
             for (int half = 0; half < 2; ++half) {
                 const int m = i * 16 + (lane >> 2) + 8 * half;
                 if (m >= rows) continue;
+                if (epilogue) {      // n is even: this thread's two columns are a (gate, up) pair
+                    const float w = pair_scale ? pair_scale[order[row0 + m]] : 1.f;
+                    if (n + 1 < N)
+                        y[(size_t)(row0 + m) * ldy + (n >> 1)] = __float2bfloat16_rn(scaled_silu_mul(acc[i][j][2 * half], acc[i][j][2 * half + 1], w));
+                    continue;
+                }
                 qi::bf16* dst = y + (size_t)(row0 + m) * ldy + n;
                 if (n < N) dst[0] = __float2bfloat16_rn(acc[i][j][2 * half]);
                 if (n + 1 < N) dst[1] = __float2bfloat16_rn(acc[i][j][2 * half + 1]);
@@ -292,48 +318,95 @@ moe_gemm_mma_kernel(const qi::bf16* __restrict__ x, const qi::bf16* __restrict__
         }
 }
 
-template <typename TY, typename TO>
+// V elements in a row: 8 (16-byte pieces) where rows and pointers allow it, else 1.
+template <typename T, int V>
+__device__ __forceinline__ void load_v(const T* p, float (&x)[V]) {
+    if constexpr (V == 8) qi::Vec8<T>::load(p, x);
+    else x[0] = qi::to_f32<T>(p[0]);
+}
+template <typename T, int V>
+__device__ __forceinline__ void store_v(T* p, float (&x)[V]) {
+    if constexpr (V == 8) qi::Vec8<T>::store(p, x);
+    else p[0] = qi::from_f32<T>(x[0]);
+}
+
+// `add` (or null): [add_parts, n, width], parts `add_stride` elements apart, added in their order after the experts.
+template <typename TY, typename TA, typename TO, int V>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const TY* __restrict__ y, const int* __restrict__ place, const float* __restrict__ weights,
-                   const TY* __restrict__ shared, TO* __restrict__ out, int n, int top, int width) {
+                   const TY* __restrict__ shared, const TA* __restrict__ add, int add_parts, size_t add_stride,
+                   TO* __restrict__ out, int n, int top, int width) {
     qi::pdl_wait();
-    const size_t total = (size_t)n * width;
+    const int pieces = width / V;
+    const size_t total = (size_t)n * pieces;
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
-        const size_t t = idx / width;
-        const int c = (int)(idx % width);
-        float acc = 0.f;
+        const size_t t = idx / pieces;
+        const int c = (int)(idx - t * pieces) * V;
+        float acc[V], v[V];
+#pragma unroll
+        for (int j = 0; j < V; ++j) acc[j] = 0.f;
         for (int k = 0; k < top; ++k) {
             const int pl = place[t * top + k];
-            if (pl >= 0 && pl < n * top) acc = fmaf(weights[t * top + k], qi::to_f32<TY>(y[(size_t)pl * width + c]), acc);
+            if (pl < 0 || pl >= n * top) continue;
+            const float w = weights ? weights[t * top + k] : 1.f;
+            load_v<TY, V>(y + (size_t)pl * width + c, v);
+#pragma unroll
+            for (int j = 0; j < V; ++j) acc[j] = fmaf(w, v[j], acc[j]);
         }
-        if (shared) acc += qi::to_f32<TY>(shared[idx]);
-        out[idx] = qi::from_f32<TO>(acc);
+        if (shared) {
+            load_v<TY, V>(shared + t * width + c, v);
+#pragma unroll
+            for (int j = 0; j < V; ++j) acc[j] += v[j];
+        }
+        if (add) {
+#pragma unroll 4
+            for (int s = 0; s < add_parts; ++s) {
+                load_v<TA, V>(add + s * add_stride + t * width + c, v);
+#pragma unroll
+                for (int j = 0; j < V; ++j) acc[j] += v[j];
+            }
+        }
+        store_v<TO, V>(out + t * width + c, acc);
     }
 }
 
-// out[i] = x[order[i] / top]: the tokens' rows in the experts' order.
-template <typename T>
+// out[i] = w x[order[i] / top]: the tokens' rows in the experts' order; w = pair_scale[order[i]], or 1 without it.
+template <typename T, int V>
 __global__ void __launch_bounds__(256)
-moe_gather_kernel(const T* __restrict__ x, const int* __restrict__ order, int top, T* __restrict__ out, int n_pairs, int n_src, int K) {
+moe_gather_kernel(const T* __restrict__ x, const int* __restrict__ order, int top, T* __restrict__ out, int n_pairs, int n_src, int K,
+                  const float* __restrict__ pair_scale) {
     qi::pdl_wait();
-    const size_t total = (size_t)n_pairs * K;
+    const int pieces = K / V;
+    const size_t total = (size_t)n_pairs * pieces;
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
-        const size_t i = idx / K;
-        const int src = order[i] / top;
-        out[idx] = (src >= 0 && src < n_src) ? x[(size_t)src * K + idx % K] : qi::from_f32<T>(0.f);
+        const size_t i = idx / pieces;
+        const int c = (int)(idx - i * pieces) * V, pair = order[i], src = pair / top;
+        float v[V];
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[j] = 0.f;
+        if (src >= 0 && src < n_src) {
+            load_v<T, V>(x + (size_t)src * K + c, v);
+            const float w = pair_scale ? pair_scale[pair] : 1.f;
+#pragma unroll
+            for (int j = 0; j < V; ++j) v[j] *= w;
+        }
+        store_v<T, V>(out + i * K + c, v);
     }
 }
 
 }  // namespace
 
+// pair_scale (or null): float32 [n_pairs] by pair; a row is multiplied by its pair's number on the way.
 extern "C" int qi_moe_gather(const void* x, int dtype, const int* order, int top, void* out, int n_pairs, int n_src, int K,
-                             cudaStream_t stream) {
+                             const float* pair_scale, cudaStream_t stream) {
     QI_REQUIRE(n_pairs >= 0 && n_src >= 0 && K > 0 && top > 0, "moe_gather: bad sizes");
     if (n_pairs == 0) return 0;
-    size_t blocks = ((size_t)n_pairs * K + 255) / 256;
+    const bool vec = K % 8 == 0 && (((uintptr_t)x | (uintptr_t)out) & 15) == 0;
+    size_t blocks = ((size_t)n_pairs * K / (vec ? 8 : 1) + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
     QI_DISPATCH_DTYPE(dtype, T, {
-        qi::launch(moe_gather_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)x, order, top, (T*)out, n_pairs, n_src, K);
+        if (vec) qi::launch(moe_gather_kernel<T, 8>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)x, order, top, (T*)out, n_pairs, n_src, K, pair_scale);
+        else qi::launch(moe_gather_kernel<T, 1>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)x, order, top, (T*)out, n_pairs, n_src, K, pair_scale);
     });
     return qi::check_launch("moe_gather");
 }
@@ -346,9 +419,11 @@ extern "C" int qi_gemm_bf16(const void* x, const void* w, void* out, int out_dty
 // w [E, N, K], y [pairs, N], all bfloat16; bounds (HOST memory) [E + 1]: expert e owns rows bounds[e] .. bounds[e + 1] - 1.
 // An expert's few hundred rows make fewer CTAs than the GPU has SMs, so the launches are dealt out over four streams
 // (the caller's and three of this library's, forked from it and joined to it by events) and run side by side; every
-// launch computes what it would alone. A stream that is being captured keeps all launches to itself.
-extern "C" int qi_moe_gemm_by_expert(const void* x, const void* w, void* y, const int* bounds, int E, int N, int K, int* status,
-                                     cudaStream_t stream) {
+// launch computes what it would alone. epilogue 1: w's rows are (gate, up) pairs and y [pairs, N / 2] = silu(gate) up. A stream that is being captured keeps all launches to itself.
+extern "C" int qi_moe_gemm_by_expert(const void* x, const void* w, void* y, const int* bounds, int E, int N, int K, int epilogue,
+                                     int* status, cudaStream_t stream) {
+    QI_REQUIRE(epilogue == 0 || (epilogue == 1 && N % 16 == 0), "moe_gemm_by_expert: unknown epilogue %d, or %d columns do not pair up", epilogue, N);
+    const int n_out = epilogue ? N / 2 : N;
     QI_REQUIRE(E > 0 && N > 0 && K > 0 && K % 8 == 0 && N % 8 == 0, "moe_gemm_by_expert: bad sizes E=%d N=%d K=%d", E, N, K);
     constexpr int kSide = 3;
     static cudaStream_t side[kSide];
@@ -382,8 +457,8 @@ extern "C" int qi_moe_gemm_by_expert(const void* x, const void* w, void* y, cons
         int swap, bn, splits;
         qi_gemm_bf16_plan(M, N, K, 0, &swap, &bn, &splits);
         const int lane = fan ? launched % (kSide + 1) : 0;
-        rc = qi_gemm_bf16((const qi::bf16*)x + (size_t)a * K, (const qi::bf16*)w + (size_t)e * N * K, (qi::bf16*)y + (size_t)a * N,
-                          qi::kBF16, M, N, K, swap, bn, 1, 0, nullptr, status, lane ? side[lane - 1] : stream);
+        rc = qi_gemm_bf16((const qi::bf16*)x + (size_t)a * K, (const qi::bf16*)w + (size_t)e * N * K, (qi::bf16*)y + (size_t)a * n_out,
+                          qi::kBF16, M, N, K, swap, bn, 1, epilogue, nullptr, status, lane ? side[lane - 1] : stream);
         ++launched;
     }
     if (fan) {    // joined also after a refusal, so that nothing of the side streams outlives the call's place in the stream
@@ -396,13 +471,14 @@ extern "C" int qi_moe_gemm_by_expert(const void* x, const void* w, void* y, cons
 
 extern "C" int qi_moe_tile_rows() { return BM; }
 
-// logits float32 [n, E]; correction float32 [E] or null; ids int32 [n, top]; weights float32 [n, top].
+// logits float32 [n, E]; correction float32 [E] or null; ids int32 [n, top]; weights float32 [n, top]. sigmoid: scores are
+// sigmoid(logit), not the softmax; normalize: the weights are divided by the chosen scores' sum.
 extern "C" int qi_moe_route(const float* logits, const float* correction, int* ids, float* weights, int n, int E, int top,
-                            float scale, cudaStream_t stream) {
+                            float scale, int sigmoid, int normalize, cudaStream_t stream) {
     QI_REQUIRE(n >= 0 && E > 0 && top > 0 && top <= E, "moe_route: bad sizes n=%d experts=%d top=%d", n, E, top);
     QI_REQUIRE(E <= 32 * kMaxPerLane, "moe_route: %d experts are above this kernel's %d", E, 32 * kMaxPerLane);
     if (n == 0) return 0;
-    qi::launch(moe_route_kernel, dim3((n + 3) / 4), dim3(128), 0, stream, logits, correction, ids, weights, n, E, top, scale);
+    qi::launch(moe_route_kernel, dim3((n + 3) / 4), dim3(128), 0, stream, logits, correction, ids, weights, n, E, top, scale, sigmoid, normalize);
     return qi::check_launch("moe_route");
 }
 
@@ -419,17 +495,20 @@ extern "C" int qi_moe_group(const int* ids, int n_pairs, int E, int tile, int ma
 }
 
 // x rows of K (ldx apart); w [E, N, K]; y [n_rows, N] (ldy apart); tiles as moe_group wrote them with tile = qi_moe_tile_rows().
-// n_src: rows of x; n_rows: rows of y (the number of (token, choice) pairs); E: experts. Tiles or source rows outside these are skipped.
+// epilogue 1: w's rows are (gate, up) pairs; y [n_rows, N / 2] = silu(s gate) s up with s = pair_scale[pair of the row] (float32
+// [n_rows] by pair) or 1 without it. n_src: rows of x; n_rows: rows of y (the number of (token, choice) pairs); E: experts. Tiles or source rows outside these are skipped.
 extern "C" int qi_moe_gemm(const void* x, int x_dtype, const void* w, int w_dtype, void* y, int y_dtype, const int* tiles,
                            int max_tiles, const int* order, int top, int gather, int N, int K, long long ldx, long long ldy,
-                           int n_src, int n_rows, int E, cudaStream_t stream) {
+                           int n_src, int n_rows, int E, int epilogue, const float* pair_scale, cudaStream_t stream) {
     QI_REQUIRE(max_tiles >= 0 && N > 0 && K > 0 && top > 0, "moe_gemm: bad sizes");
-    QI_REQUIRE(ldx >= K && ldy >= N, "moe_gemm: a leading dimension is smaller than its row");
+    QI_REQUIRE((epilogue == 0 && !pair_scale) || (epilogue == 1 && N % 2 == 0), "moe_gemm: unknown epilogue %d, or %d columns do not pair up", epilogue, N);
+    QI_REQUIRE(ldx >= K && ldy >= (epilogue ? N / 2 : N), "moe_gemm: a leading dimension is smaller than its row");
     QI_REQUIRE(max_tiles <= 65535, "moe_gemm: %d row tiles are too many for one launch", max_tiles);
     if (max_tiles == 0) return 0;
     if (x_dtype == qi::kBF16 && w_dtype == qi::kBF16 && y_dtype == qi::kBF16 && K % 8 == 0 && ldx % 8 == 0) {
         qi::launch(moe_gemm_mma_kernel, dim3((N + MN - 1) / MN, max_tiles), dim3(128), 0, stream, (const qi::bf16*)x,
-                   (const qi::bf16*)w, (qi::bf16*)y, tiles, order, top, gather, N, K, ldx, ldy, n_src, n_rows, E);
+                   (const qi::bf16*)w, (qi::bf16*)y, tiles, order, top, gather, N, K, ldx, ldy, n_src, n_rows, E, epilogue,
+                   pair_scale);
         return qi::check_launch("moe_gemm_mma");
     }
     const dim3 grid((N + BN - 1) / BN, max_tiles), block(256);
@@ -437,25 +516,38 @@ extern "C" int qi_moe_gemm(const void* x, int x_dtype, const void* w, int w_dtyp
         QI_DISPATCH_DTYPE(w_dtype, TW, {
             QI_DISPATCH_DTYPE(y_dtype, TY, {
                 qi::launch(moe_gemm_kernel<TX, TW, TY>, grid, block, 0, stream, (const TX*)x, (const TW*)w, (TY*)y, tiles, order, top,
-                           gather, N, K, ldx, ldy, n_src, n_rows, E);
+                           gather, N, K, ldx, ldy, n_src, n_rows, E, epilogue, pair_scale);
             });
         });
     });
     return qi::check_launch("moe_gemm");
 }
 
-// y [n * top, width] in y_dtype (sorted rows); place int32 [n, top]; weights float32 [n, top]; shared [n, width] in y_dtype or null.
-extern "C" int qi_moe_combine(const void* y, int y_dtype, const int* place, const float* weights, const void* shared, void* out,
-                              int out_dtype, int n, int top, int width, cudaStream_t stream) {
+// y [n * top, width] in y_dtype (sorted rows); place int32 [n, top]; weights float32 [n, top] or null (1); shared [n, width] in
+// y_dtype or null; add (or null): another output of the same tokens, [add_parts, n, width] in add_dtype, parts add_stride elements apart.
+extern "C" int qi_moe_combine(const void* y, int y_dtype, const int* place, const float* weights, const void* shared, const void* add,
+                              int add_dtype, int add_parts, long long add_stride, void* out, int out_dtype, int n, int top, int width,
+                              cudaStream_t stream) {
+    QI_REQUIRE(!add || (add_parts >= 1 && (add_parts == 1 || add_stride >= (long long)n * width)), "moe_combine: the parts to add overlap");
     QI_REQUIRE(n >= 0 && top > 0 && width > 0, "moe_combine: bad sizes");
     if (n == 0) return 0;
-    size_t blocks = ((size_t)n * width + 255) / 256;
+    const bool vec = width % 8 == 0 && add_stride % 8 == 0 &&
+                     (((uintptr_t)y | (uintptr_t)shared | (uintptr_t)add | (uintptr_t)out) & 15) == 0;
+    const int threads = vec && (size_t)n * width / 8 < 148 * 256 ? 64 : 256;       // few tokens: more and smaller blocks
+    size_t blocks = ((size_t)n * width / (vec ? 8 : 1) + threads - 1) / threads;
     if (blocks > 148 * 16) blocks = 148 * 16;
+    if (!add) add_dtype = y_dtype;
+#define QI_COMBINE(V)                                                                                                            \
+    qi::launch(moe_combine_kernel<TY, TA, TO, V>, dim3((unsigned)blocks), dim3(threads), 0, stream, (const TY*)y, place, weights, \
+               (const TY*)shared, (const TA*)add, add_parts, (size_t)add_stride, (TO*)out, n, top, width)
     QI_DISPATCH_DTYPE(y_dtype, TY, {
-        QI_DISPATCH_DTYPE(out_dtype, TO, {
-            qi::launch(moe_combine_kernel<TY, TO>, dim3((unsigned)blocks), dim3(256), 0, stream, (const TY*)y, place, weights,
-                       (const TY*)shared, (TO*)out, n, top, width);
+        QI_DISPATCH_DTYPE(add_dtype, TA, {
+            QI_DISPATCH_DTYPE(out_dtype, TO, {
+                if (vec) QI_COMBINE(8);
+                else QI_COMBINE(1);
+            });
         });
     });
+#undef QI_COMBINE
     return qi::check_launch("moe_combine");
 }

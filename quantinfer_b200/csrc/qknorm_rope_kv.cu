@@ -303,8 +303,9 @@ extern "C" int qi_qk_norm_rope_kv(const void* qkv, int qkv_splits, void* q_out, 
 // (k_pages [pages, nkv, page_size, d], v_pages [pages, nkv, page_size, dv]; null: nothing is written).
 // Options for designs that ask for them: one RMS norm over the whole of q and one over the whole of k (all heads
 // at once, gain per coordinate) before the rotation, or one over every head by itself (`head_norm`; a gain of d numbers
-// that the heads share); values that are the keys as projected (no v in the row); and a factor on q that grows with the
-// position, 1 + temp_coef ln(floor((p + 1) / temp_every) + 1).
+// that the heads share); values that are the keys as projected (no v in the row); a factor on q that grows with the
+// position, 1 + temp_coef ln(floor((p + 1) / temp_every) + 1); and values mixed with another layer's values of the same
+// token (`v_first`, rows `ldv` elements apart): v <- (1 - v_share) v + v_share v_first, in 32-bit.
 namespace {
 
 __device__ __forceinline__ float query_factor(int pos, float temp_coef, int temp_every) {
@@ -318,7 +319,8 @@ bias_rope_kv_kernel(const T* __restrict__ proj, long long ld, const float* __res
                     const int* __restrict__ token_req, const int* __restrict__ block_table, int max_blocks, int page_size,
                     int num_pages, T* __restrict__ k_pages, T* __restrict__ v_pages, int nq, int nkv, int d, int dv,
                     const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps, int head_norm, int v_from_k,
-                    float temp_coef, int temp_every, int* __restrict__ status) {
+                    float temp_coef, int temp_every, const T* __restrict__ v_first, long long ldv, float v_share,
+                    int* __restrict__ status) {
     __shared__ float scratch[32];
     extern __shared__ float head_inv[];         // [nq + nkv] with norms of every head by itself
     qi::pdl_wait();
@@ -373,9 +375,10 @@ bias_rope_kv_kernel(const T* __restrict__ proj, long long ld, const float* __res
     const int half = rot / 2;
     const float q_factor = query_factor(pos, temp_coef, temp_every);
     for (int e = threadIdx.x; e < total; e += blockDim.x) {
-        if (e >= qk) {   // a value: bias only
+        if (e >= qk) {   // a value: bias, and another layer's value mixed in
             const int hv = (e - qk) / dv, i = (e - qk) % dv;
-            const float v = qi::to_f32<T>(row[e]) + (bias ? bias[e] : 0.f);
+            float v = qi::to_f32<T>(row[e]) + (bias ? bias[e] : 0.f);
+            if (v_first) v = (1.f - v_share) * v + v_share * qi::to_f32<T>(v_first[(size_t)t * ldv + (e - qk)]);
             if (vrow) vrow[(size_t)hv * page_size * dv + i] = qi::from_f32<T>(v);
             continue;
         }
@@ -398,14 +401,16 @@ bias_rope_kv_kernel(const T* __restrict__ proj, long long ld, const float* __res
     }
 }
 
-// The form for rows without biases, rotation and values from keys, in 16-byte pieces: LANES lanes a head (eight coordinates
-// each, d <= 8 LANES), every operand read once. A warp takes 32 / LANES heads of q, k and v in turn.
+// The form for rows without biases and values from keys, in 16-byte pieces: LANES lanes a head (eight coordinates each, d <=
+// 8 LANES), every operand read once. A warp takes 32 / LANES heads of q, k and v in turn. Norms of every head by itself, a
+// rotation in neighbouring pairs (a lane holds whole pairs) and values mixed with another layer's are each optional.
 template <typename T, int LANES>
 __global__ void __launch_bounds__(256)
-head_norm_kv_kernel(const T* __restrict__ proj, long long ld, T* __restrict__ q_out, const int* __restrict__ positions,
+head_rope_kv_kernel(const T* __restrict__ proj, long long ld, T* __restrict__ q_out, const int* __restrict__ positions,
                     const int* __restrict__ token_req, const int* __restrict__ block_table, int max_blocks, int page_size,
                     int num_pages, T* __restrict__ k_pages, T* __restrict__ v_pages, int nq, int nkv, int d, int dv,
                     const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps, float temp_coef, int temp_every,
+                    const float* __restrict__ inv_freq, int rot, const T* __restrict__ v_first, long long ldv, float v_share,
                     int n_tokens, int* __restrict__ status) {
     qi::pdl_wait();
     const int heads = nq + 2 * nkv, per_block = 256 / LANES;
@@ -445,11 +450,33 @@ head_norm_kv_kernel(const T* __restrict__ proj, long long ld, T* __restrict__ q_
             dst = (is_v ? v_pages : k_pages) + (((size_t)page * nkv + g) * page_size + pos % page_size) * (size_t)width;
         }
         if (!is_v) {
-            float g[8];
-            qi::Vec8<float>::load((hd < nq ? q_gain : k_gain) + i, g);
-            const float inv = 1.0f / sqrtf(sq / (float)d + eps) * (hd < nq ? query_factor(pos, temp_coef, temp_every) : 1.f);
+            const float factor = hd < nq ? query_factor(pos, temp_coef, temp_every) : 1.f;
+            if (q_gain) {
+                float g[8];
+                qi::Vec8<float>::load((hd < nq ? q_gain : k_gain) + i, g);
+                const float inv = 1.0f / sqrtf(sq / (float)d + eps);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) x[j] = x[j] * inv * g[j];
+                for (int j = 0; j < 8; ++j) x[j] = x[j] * inv * g[j];
+            }
+#pragma unroll
+            for (int j = 0; j < 8; j += 2) {
+                if (i + j < rot) {
+                    float sn, cs;
+                    sincosf((float)pos * inv_freq[(i + j) >> 1], &sn, &cs);
+                    const float u = x[j], v = x[j + 1];
+                    x[j] = u * cs - v * sn;
+                    x[j + 1] = v * cs + u * sn;
+                }
+            }
+            if (temp_every > 0) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) x[j] *= factor;
+            }
+        } else if (v_first) {
+            float f[8];
+            qi::Vec8<T>::load(v_first + (size_t)t * ldv + (size_t)(hd - nq - nkv) * dv + i, f);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) x[j] = (1.f - v_share) * x[j] + v_share * f[j];
         }
         qi::Vec8<T>::store(dst + i, x);
     }
@@ -459,13 +486,15 @@ head_norm_kv_kernel(const T* __restrict__ proj, long long ld, T* __restrict__ q_
 
 // q_gain, k_gain (both or neither; float32 [nq d], [nkv d]): q as a whole and k as a whole each pass an RMS norm with that
 // gain and `eps` before the rotation; with head_norm every head by itself does, with a gain of d numbers that the heads
-// share. temp_every > 0: q is multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1). v_from_k: the rows hold no v; a position's value is its key as projected (dv = d).
+// share. temp_every > 0: q is multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1). v_first (or null; rows `ldv`
+// elements apart, in `dtype`): a value v becomes (1 - v_share) v + v_share v_first before it is cached. v_from_k: the rows hold no v; a position's value is its key as projected (dv = d).
 extern "C" int qi_norm_rope_kv_ex(const void* proj, long long ld, const float* bias, void* q_out, int dtype,
                                const float* inv_freq, int rot, int interleaved, const int* positions,
                                const int* token_req, const int* block_table, int max_blocks, int page_size,
                                int num_pages, void* k_pages, void* v_pages, int n_tokens, int nq, int nkv, int d,
                                int dv, const float* q_gain, const float* k_gain, float eps, int head_norm, int v_from_k, float temp_coef,
-                               int temp_every, int* status, cudaStream_t stream) {
+                               int temp_every, const void* v_first, long long ldv, float v_share, int* status, cudaStream_t stream) {
+    QI_REQUIRE(!v_first || (!v_from_k && ldv >= (long long)nkv * dv), "bias_rope_kv: values to mix in need rows of values");
     QI_REQUIRE(n_tokens >= 0 && nq > 0 && nkv > 0 && d > 0 && dv > 0, "bias_rope_kv: bad sizes");
     QI_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= d, "bias_rope_kv: %d rotated coordinates do not fit a head of %d", rot, d);
     QI_REQUIRE(rot == 0 || inv_freq, "bias_rope_kv: a rotation needs its inverse frequencies");
@@ -476,16 +505,16 @@ extern "C" int qi_norm_rope_kv_ex(const void* proj, long long ld, const float* b
     QI_REQUIRE(!k_pages || (block_table && max_blocks > 0 && page_size > 0 && num_pages > 0), "bias_rope_kv: bad page geometry");
     QI_REQUIRE(nq + nkv <= 8192, "bias_rope_kv: too many heads");
     if (n_tokens == 0) return 0;
-    if (q_gain && head_norm && !bias && !rot && !v_from_k && d % 8 == 0 && dv % 8 == 0 && d <= 256 && dv <= 256 && ld % 8 == 0 &&
-        (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)q_gain | (uintptr_t)k_gain) & 15) == 0) {
+    if ((!q_gain || head_norm) && !bias && (!rot || interleaved) && !v_from_k && d % 8 == 0 && dv % 8 == 0 && d <= 256 && dv <= 256 && ld % 8 == 0 && ldv % 8 == 0 &&
+        (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)q_gain | (uintptr_t)k_gain | (uintptr_t)v_first) & 15) == 0) {
         const int wide = d > dv ? d : dv;
         const int lanes = wide <= 32 ? 4 : wide <= 64 ? 8 : wide <= 128 ? 16 : 32, per_block = 256 / lanes;
         long long blocks = ((long long)n_tokens * (nq + 2 * nkv) + per_block - 1) / per_block;
         if (blocks > 148 * 64) blocks = 148 * 64;
 #define QI_HN(L)                                                                                                                     \
-    qi::launch(head_norm_kv_kernel<T, L>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)proj, ld, (T*)q_out, positions, token_req, \
+    qi::launch(head_rope_kv_kernel<T, L>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)proj, ld, (T*)q_out, positions, token_req, \
                block_table, max_blocks, page_size, num_pages, (T*)k_pages, (T*)v_pages, nq, nkv, d, dv, q_gain, k_gain, eps, temp_coef, \
-               temp_every, n_tokens, status)
+               temp_every, inv_freq, rot, (const T*)v_first, ldv, v_share, n_tokens, status)
         QI_DISPATCH_DTYPE(dtype, T, {
             if (lanes == 4) QI_HN(4);
             else if (lanes == 8) QI_HN(8);
@@ -493,12 +522,13 @@ extern "C" int qi_norm_rope_kv_ex(const void* proj, long long ld, const float* b
             else QI_HN(32);
         });
 #undef QI_HN
-        return qi::check_launch("head_norm_kv");
+        return qi::check_launch("head_rope_kv");
     }
     QI_DISPATCH_DTYPE(dtype, T, {
         qi::launch(bias_rope_kv_kernel<T>, dim3(n_tokens), dim3(256), head_norm ? sizeof(float) * (nq + nkv) : 0, stream, (const T*)proj, ld, bias, (T*)q_out, inv_freq, rot,
                    interleaved, positions, token_req, block_table, max_blocks, page_size, num_pages, (T*)k_pages, (T*)v_pages,
-                   nq, nkv, d, dv, q_gain, k_gain, eps, head_norm, v_from_k, temp_coef, temp_every, status);
+                   nq, nkv, d, dv, q_gain, k_gain, eps, head_norm, v_from_k, temp_coef, temp_every,
+                   (const T*)v_first, ldv, v_share, status);
     });
     return qi::check_launch("bias_rope_kv");
 }
@@ -509,5 +539,5 @@ extern "C" int qi_bias_rope_kv(const void* proj, long long ld, const float* bias
                                int num_pages, void* k_pages, void* v_pages, int n_tokens, int nq, int nkv, int d,
                                int dv, int* status, cudaStream_t stream) {
     return qi_norm_rope_kv_ex(proj, ld, bias, q_out, dtype, inv_freq, rot, interleaved, positions, token_req, block_table, max_blocks,
-                           page_size, num_pages, k_pages, v_pages, n_tokens, nq, nkv, d, dv, nullptr, nullptr, 0.f, 0, 0, 0.f, 0, status, stream);
+                           page_size, num_pages, k_pages, v_pages, n_tokens, nq, nkv, d, dv, nullptr, nullptr, 0.f, 0, 0, 0.f, 0, nullptr, 0, 0.f, status, stream);
 }

@@ -25,7 +25,7 @@ STATUS_NON_FINITE = 4
 STATUS_WAIT_TIMEOUT = 8
 STATUS_BAD_RANGE = 16
 
-ABI_VERSION = 15
+ABI_VERSION = 16
 
 
 def status_names(code: int) -> list:
@@ -467,14 +467,15 @@ def _req_bias(bias, nq: int) -> None:
 
 def attention_generic(q, out, k_pages, v_pages, block_table, positions, token_req, nq, nkv, d,
                       scale: float, window: int, status, chunk: int = 0, gate=None, softcap: float = 0.0,
-                      out_scale: float = 1.0, sink=None, bias=None) -> None:
+                      out_scale: float = 1.0, sink=None, bias=None, keep_first: int = 0) -> None:
     """Causal paged GQA attention, 32-bit arithmetic, any span length and page size. `sink` (float32 [nq] or None): the
     softmax's denominator of head h holds exp(sink[h]) once more, with no key and no value. Values may have another
     size than keys (v_pages [pages, nkv, page_size, dv], out [n, nq dv]); `chunk` > 0: a query sees only the keys
     of its own chunk of that many positions (counted from the sequence's start); `gate` [n, >= nq dv] (a view whose
     rows may lie further apart): the result is multiplied by sigmoid(gate). `softcap` c > 0: a score s becomes
     c tanh(s / c) before the softmax. `out_scale` multiplies the result. `bias` (float32 [nq, reach] or None): a key n
-    positions back adds bias[h, min(n, reach - 1)] to its score (after the cap)."""
+    positions back adds bias[h, min(n, reach - 1)] to its score (after the cap). The sequence's first `keep_first` keys
+    stay visible behind a window or a chunk."""
     _req_bias(bias, nq)
     _req(q, "q", ndim=2)
     _req(k_pages, "k_pages", q.dtype, 4)
@@ -502,7 +503,7 @@ def attention_generic(q, out, k_pages, v_pages, block_table, positions, token_re
           _ptr(q), _ptr(out), _code(q), _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
         block_table.shape[1], k_pages.shape[2], k_pages.shape[0], _ptr(positions), _ptr(token_req), n,
         nq, nkv, d, dv, C.c_float(scale), C.c_float(softcap or 0.0), C.c_float(out_scale), int(window or 0), int(chunk or 0), _ptr(gate), C.c_longlong(ldg), _ptr(sink),
-        _ptr(bias), bias.shape[1] if bias is not None else 0, C.c_longlong(ldo), _ptr(status), _stream())
+        _ptr(bias), bias.shape[1] if bias is not None else 0, C.c_longlong(ldo), int(keep_first or 0), _ptr(status), _stream())
 
 
 def attention_mma_supported(nq: int, nkv: int, d: int) -> bool:
@@ -550,7 +551,7 @@ def attention_prefill_ranges(n_ctas: int, max_kv_len: int) -> int:
 def attention_prefill(q, out, k_pages, v_pages, block_table, q_start, start_pos, tile_req, tile_q0,
                       nq, nkv, d, scale: float, window: int, status, use_tma: bool | None = None,
                       impl: str | None = None, max_kv_len: int = 0, key_ranges: int | None = None, chunk: int = 0,
-                      gate=None, softcap: float = 0.0, out_scale: float = 1.0, sink=None, bias=None) -> None:
+                      gate=None, softcap: float = 0.0, out_scale: float = 1.0, sink=None, bias=None, keep_first: int = 0) -> None:
     """Causal paged GQA flash attention (bfloat16, head size 64 or 128) for spans of any
     length. `tile_req[i]`, `tile_q0[i]`: request index and first flat token of the i-th
     block of up to QUERY_TILE query rows.
@@ -565,7 +566,8 @@ def attention_prefill(q, out, k_pages, v_pages, block_table, q_start, start_pos,
     start), `gate` (bfloat16 [n, nq d], rows a multiple of 8 elements apart and 16-byte aligned: the output is
     multiplied with its sigmoid), `softcap` c > 0 (a score s becomes c tanh(s / c)), `out_scale` (a factor on the
     result), `sink` (float32 [nq]: exp(sink[h]) once more in the softmax's denominator of head h) and `bias` (float32
-    [nq, reach]: a key n positions back adds bias[h, min(n, reach - 1)] to its score)."""
+    [nq, reach]: a key n positions back adds bias[h, min(n, reach - 1)] to its score) and `keep_first` (the sequence's
+    first keys that stay visible behind a window or a chunk)."""
     _req_bias(bias, nq)
     if impl is None and use_tma is not None:
         impl = "tma" if use_tma else "cpasync"
@@ -606,10 +608,11 @@ def attention_prefill(q, out, k_pages, v_pages, block_table, q_start, start_pos,
             k_pages.shape[2], k_pages.shape[0], _ptr(q_start), _ptr(start_pos), _ptr(tile_req), _ptr(tile_q0),
             tile_req.numel(), q.shape[0], nq, nkv, d, C.c_float(scale), int(window or 0), int(chunk or 0), _ptr(gate),
             C.c_longlong(ldg), ranges, _ptr(ws), _ptr(status), C.c_float(softcap or 0.0), C.c_float(out_scale), _ptr(sink),
-            _ptr(bias), bias.shape[1] if bias is not None else 0, C.c_longlong(ldo), _stream())
+            _ptr(bias), bias.shape[1] if bias is not None else 0, C.c_longlong(ldo), int(keep_first or 0), _stream())
         return
-    if chunk or gate is not None or softcap or out_scale != 1.0 or sink is not None or bias is not None:
-        raise KernelError(f"attention_prefill: the {impl!r} kernel takes neither a chunk bound, a gate, a soft cap, an output factor, a sink nor a bias")
+    if chunk or gate is not None or softcap or out_scale != 1.0 or sink is not None or bias is not None or keep_first:
+        raise KernelError(f"attention_prefill: the {impl!r} kernel takes neither a chunk bound, a gate, a soft cap, an output factor, a sink, a bias "
+                          "nor kept first keys")
     _req(out, "out", torch.bfloat16, 2)
     if impl not in ("tma", "cpasync"):
         raise KernelError(f"attention_prefill: unknown kernel {impl!r}")
@@ -1128,6 +1131,33 @@ def latent_prepare(proj, kv_offset, q_out, gain, eps: float, inv_freq, rot_dims:
           C.c_float(magnitude), _ptr(status), _stream())
 
 
+def latent_down(proj, q_rank: int, q_gain, cq, gain, eps: float, inv_freq, rot_dims: int, positions, token_req, block_table, cache,
+                r: int, rank: int, status, half_split: bool = False, magnitude: float = 1.0) -> None:
+    """From the projection's rows [query latent (q_rank) | latent (rank) | rotated key part (r)], whole [n, q_rank + rank + r] or
+    as partial sums [parts, n, ...]: the query latent over its root mean square times q_gain goes to cq [n, q_rank]; the
+    rest is normalised, rotated and cached as `latent_prepare` does."""
+    _req(proj, "proj")
+    _req(cq, "cq", ndim=2)
+    n, width = proj.shape[-2], proj.shape[-1]
+    if proj.dim() not in (2, 3) or width != q_rank + rank + r or tuple(cq.shape) != (n, q_rank):
+        raise KernelError(f"latent_down: proj {tuple(proj.shape)} / cq {tuple(cq.shape)} do not fit {q_rank} + {rank} + {r}")
+    _req(q_gain, "q_gain", torch.float32, 1)
+    _req(gain, "gain", torch.float32, 1)
+    _req(cache, "cache", cq.dtype, 3)
+    _req(block_table, "block_table", torch.int32, 2)
+    _req(positions, "positions", torch.int32, 1)
+    _req(token_req, "token_req", torch.int32, 1)
+    if rot_dims:
+        _req(inv_freq, "inv_freq", torch.float32, 1)
+    if cache.shape[2] != rank + r or gain.numel() != rank or q_gain.numel() != q_rank or (rot_dims and inv_freq.numel() * 2 != rot_dims):
+        raise KernelError(f"latent_down: cache {tuple(cache.shape)}, gains or frequencies do not fit {q_rank} / {rank} + {r}")
+    parts = proj.shape[0] if proj.dim() == 3 else 1
+    _call("rope", "latent_down", library().qi_latent_down, _ptr(proj), _code(proj), parts, C.c_longlong(n * width), C.c_longlong(width),
+          q_rank, _ptr(q_gain), _ptr(cq), _code(cq), _ptr(gain), C.c_float(eps), _ptr(inv_freq if rot_dims else None), rot_dims,
+          _ptr(positions), _ptr(token_req), _ptr(block_table), block_table.shape[1], cache.shape[1], cache.shape[0], _ptr(cache), n, r,
+          rank, int(bool(half_split)), C.c_float(magnitude), _ptr(status), _stream())
+
+
 def latent_attention_generic(q, out, cache, sink, block_table, positions, token_req, scale: float, window: int, status) -> None:
     """Causal attention of every head over one shared cached row per position: q [n, heads, W], cache [pages,
     page_size, W], out [n, heads, R] = sum_j p_j cache[j, :R]; the softmax's denominator also holds exp(sink[h])
@@ -1260,7 +1290,7 @@ def concat_cast(a, b, out) -> None:
 
 def bias_rope_kv(proj, bias, q_out, inv_freq, rot: int, interleaved: bool, positions, token_req, block_table, page_size: int,
                  k_pages, v_pages, nq: int, nkv: int, d: int, dv: int, status, q_gain=None, k_gain=None, norm_eps: float = 0.0,
-                 values_from_keys: bool = False, head_norm: bool = False, q_temp=None) -> None:
+                 values_from_keys: bool = False, head_norm: bool = False, q_temp=None, v_first=None, v_share: float = 0.0) -> None:
     """proj [n, >= (nq + nkv) d + nkv dv] holds q | k | v (more columns may follow); bias float32 over those columns or
     None; the first `rot` coordinates of each q and k head turn by position * inv_freq[pair] (computed here in 32-bit:
     no table, no limit on positions); q goes to q_out [n, nq d], k and v into the pages (None: nothing is written).
@@ -1268,7 +1298,8 @@ def bias_rope_kv(proj, bias, q_out, inv_freq, rot: int, interleaved: bool, posit
     and `norm_eps` before the rotation. values_from_keys: the rows hold no v; a position's value is its key as
     projected, before norm and rotation (dv = d). head_norm: every head of q and k passes an RMS norm of its own instead, with
     gains q_gain, k_gain [d] that the heads share. q_temp (coef, every) or None: q is multiplied by
-    1 + coef ln(floor((p + 1) / every) + 1) at position p."""
+    1 + coef ln(floor((p + 1) / every) + 1) at position p. v_first [n, nkv dv] (maybe a block of columns of wider rows) or
+    None: a value v is cached as (1 - v_share) v + v_share v_first."""
     if not proj.is_cuda or proj.dim() != 2 or proj.stride(1) != 1:
         raise KernelError("bias_rope_kv: proj must be a CUDA tensor with contiguous rows")
     _req(q_out, "q_out", proj.dtype, 2)
@@ -1293,6 +1324,10 @@ def bias_rope_kv(proj, bias, q_out, inv_freq, rot: int, interleaved: bool, posit
             raise KernelError("bias_rope_kv: one inverse frequency a pair")
     _req(positions, "positions", torch.int32, 1)
     _req(token_req, "token_req", torch.int32, 1)
+    if v_first is not None:
+        _cols(v_first, "v_first", proj.dtype)
+        if values_from_keys or tuple(v_first.shape) != (n, nkv * dv):
+            raise KernelError(f"bias_rope_kv: values to mix in of shape {tuple(v_first.shape)} for {nkv} value heads of {dv}")
     num_pages = max_blocks = 0
     if k_pages is not None:
         _req(k_pages, "k_pages", proj.dtype, 4)
@@ -1305,7 +1340,8 @@ def bias_rope_kv(proj, bias, q_out, inv_freq, rot: int, interleaved: bool, posit
           _code(proj), _ptr(inv_freq if rot else None), rot, int(bool(interleaved)), _ptr(positions), _ptr(token_req),
           _ptr(block_table), max_blocks, page_size, num_pages, _ptr(k_pages), _ptr(v_pages), n, nq, nkv, d, dv, _ptr(q_gain),
           _ptr(k_gain), C.c_float(norm_eps), int(bool(head_norm)), int(bool(values_from_keys)), C.c_float(q_temp[0] if q_temp else 0.0),
-          int(q_temp[1]) if q_temp else 0, _ptr(status), _stream())
+          int(q_temp[1]) if q_temp else 0, _ptr(v_first), C.c_longlong(v_first.stride(0) if v_first is not None else 0), C.c_float(v_share),
+          _ptr(status), _stream())
 
 
 def ssm_scan(xbc, raw_dt, dt_bias, a_log, d_skip, state, y, q_start, start_pos, slot_ids, heads: int, groups: int, P: int, N: int,
@@ -1588,13 +1624,15 @@ def moe_tile_rows() -> int:
     return int(library().qi_moe_tile_rows())
 
 
-def moe_route(logits, correction, ids, weights, scale: float) -> None:
-    """Per token: softmax over all experts, the `top` largest of softmax + correction, weights = the chosen experts' softmax
-    over their sum, times scale. logits float32 [n, E]; ids int32 [n, top]; weights float32 [n, top]."""
+def moe_route(logits, correction, ids, weights, scale: float, scoring: str = "softmax", normalize: bool = True) -> None:
+    """Per token: scores = softmax over all experts (or the sigmoid of each logit: `scoring` "sigmoid"), the `top` largest of
+    score + correction, weights = the chosen experts' scores over their sum (as they are without `normalize`), times scale. logits float32 [n, E]; ids int32 [n, top]; weights float32 [n, top]."""
     _req(logits, "logits", torch.float32, 2)
     _req(ids, "ids", torch.int32, 2)
     _req(weights, "weights", torch.float32, 2)
     n, E = logits.shape
+    if scoring not in ("softmax", "sigmoid"):
+        raise KernelError(f"moe_route: unknown scores {scoring!r}")
     if ids.shape != weights.shape or ids.shape[0] != n:
         raise KernelError("moe_route: shapes do not agree")
     if correction is not None:
@@ -1602,7 +1640,7 @@ def moe_route(logits, correction, ids, weights, scale: float) -> None:
         if correction.numel() != E:
             raise KernelError("moe_route: one correction an expert")
     _call("gemm", "moe_route", library().qi_moe_route, _ptr(logits), _ptr(correction), _ptr(ids), _ptr(weights), n, E,
-          ids.shape[1], C.c_float(scale), _stream())
+          ids.shape[1], C.c_float(scale), int(scoring == "sigmoid"), int(bool(normalize)), _stream())
 
 
 def moe_group(ids, n_experts: int, offsets, order, place, tiles) -> None:
@@ -1617,61 +1655,88 @@ def moe_group(ids, n_experts: int, offsets, order, place, tiles) -> None:
           _ptr(order), _ptr(place), _ptr(tiles), _stream())
 
 
-def moe_gemm(x, w, y, tiles, order, top: int, gather: bool) -> None:
-    """y[i] = w[expert of sorted row i] . x[order[i] // top if gather else i]. x [rows, K]; w [E, N, K]; y [pairs, N]."""
+def moe_gemm(x, w, y, tiles, order, top: int, gather: bool, epilogue: str | None = None, pair_scale=None) -> None:
+    """y[i] = w[expert of sorted row i] . x[order[i] // top if gather else i]. x [rows, K]; w [E, N, K]; y [pairs, N].
+    epilogue "silu_mul": w's rows are (gate, up) pairs and y [pairs, N / 2] = silu(s gate) (s up), s = pair_scale[order[i]]
+    (float32 [pairs]) or 1 without it."""
     _req(x, "x", ndim=2)
     _req(w, "w", ndim=3)
     _req(y, "y", ndim=2)
     _req(tiles, "tiles", torch.int32, 2)
     _req(order, "order", torch.int32)
     N, K = w.shape[1], w.shape[2]
-    if x.shape[1] != K or y.shape[1] != N:
+    _moe_epilogue("moe_gemm", epilogue, pair_scale, order)
+    n_out = N // 2 if epilogue else N
+    if x.shape[1] != K or y.shape[1] != n_out:
         raise KernelError(f"moe_gemm: shapes do not agree: x {tuple(x.shape)}, w {tuple(w.shape)}, y {tuple(y.shape)}")
     _call("gemm", "moe_gemm", library().qi_moe_gemm, _ptr(x), _code(x), _ptr(w), _code(w), _ptr(y), _code(y), _ptr(tiles),
-          tiles.shape[0], _ptr(order), top, int(bool(gather)), N, K, C.c_longlong(K), C.c_longlong(N), x.shape[0], y.shape[0],
-          w.shape[0], _stream())
+          tiles.shape[0], _ptr(order), top, int(bool(gather)), N, K, C.c_longlong(K), C.c_longlong(n_out), x.shape[0], y.shape[0],
+          w.shape[0], int(epilogue is not None), _ptr(pair_scale), _stream())
 
 
-def moe_gather(x, order, top: int, out) -> None:
-    """out[i] = x[order[i] // top]: the tokens' rows in the experts' order. x [n, K]; out [pairs, K]."""
+def _moe_epilogue(name: str, epilogue, pair_scale, order) -> None:
+    if epilogue not in (None, "silu_mul") or (pair_scale is not None and epilogue is None):
+        raise KernelError(f"{name}: unknown epilogue {epilogue!r}, or pair weights without one")
+    if pair_scale is not None:
+        _req(pair_scale, "pair_scale", torch.float32)
+        if pair_scale.numel() != order.numel():
+            raise KernelError(f"{name}: one weight a (token, choice) pair")
+
+
+def moe_gather(x, order, top: int, out, pair_scale=None) -> None:
+    """out[i] = x[order[i] // top]: the tokens' rows in the experts' order, times pair_scale[order[i]] (float32 [pairs]) when
+    given. x [n, K]; out [pairs, K]."""
     _req(x, "x", ndim=2)
     _req(out, "out", x.dtype, 2)
     _req(order, "order", torch.int32)
     if out.shape[1] != x.shape[1] or order.numel() != out.shape[0]:
         raise KernelError("moe_gather: shapes do not agree")
+    _moe_epilogue("moe_gather", "silu_mul", pair_scale, order)
     _call("gemm", "moe_gather", library().qi_moe_gather, _ptr(x), _code(x), _ptr(order), top, _ptr(out), out.shape[0], x.shape[0],
-          x.shape[1], _stream())
+          x.shape[1], _ptr(pair_scale), _stream())
 
 
-def moe_gemm_by_expert(x, w, y, bounds, status) -> None:
+def moe_gemm_by_expert(x, w, y, bounds, status, epilogue: str | None = None) -> None:
     """y[rows of expert e] = x[rows of expert e] . w[e]^T through the tcgen05 product, one launch an expert. x [pairs, K]
-    in the experts' order, w [E, N, K], y [pairs, N], bfloat16; bounds: E + 1 ascending row numbers, on the HOST."""
+    in the experts' order, w [E, N, K], y [pairs, N], bfloat16; bounds: E + 1 ascending row numbers, on the HOST. epilogue
+    "silu_mul": w's rows are (gate, up) pairs and y [pairs, N / 2] = silu(gate) up."""
     _req(x, "x", torch.bfloat16, 2)
     _req(w, "w", torch.bfloat16, 3)
     _req(y, "y", torch.bfloat16, 2)
     E, N, K = w.shape
-    if x.shape[1] != K or y.shape[1] != N or x.shape[0] != y.shape[0] or len(bounds) != E + 1 or bounds[-1] > x.shape[0]:
+    _moe_epilogue("moe_gemm_by_expert", epilogue, None, None)
+    if x.shape[1] != K or y.shape[1] != (N // 2 if epilogue else N) or x.shape[0] != y.shape[0] or len(bounds) != E + 1 or bounds[-1] > x.shape[0]:
         raise KernelError("moe_gemm_by_expert: shapes do not agree")
     arr = (C.c_int * (E + 1))(*bounds)
-    _call("gemm", "moe_gemm_by_expert", library().qi_moe_gemm_by_expert, _ptr(x), _ptr(w), _ptr(y), arr, E, N, K, _ptr(status), _stream())
+    _call("gemm", "moe_gemm_by_expert", library().qi_moe_gemm_by_expert, _ptr(x), _ptr(w), _ptr(y), arr, E, N, K, int(epilogue is not None),
+          _ptr(status), _stream())
 
 
-def moe_combine(y, place, weights, shared, out) -> None:
-    """out[t] = sum_k weights[t, k] * y[place[t, k]] (+ shared[t]). y [n top, width]; out [n, width]."""
+def moe_combine(y, place, weights, shared, out, add=None, top: int | None = None) -> None:
+    """out[t] = sum_k weights[t, k] * y[place[t, k]] (+ shared[t]) (+ add[t]). y [n top, width]; out [n, width]. weights None: the
+    plain sum over `top` choices. add: another output of the same tokens, [n, width] or the partial sums [parts, n, width] of
+    a product whose contraction was cut, added in their order."""
     _req(y, "y", ndim=2)
     _req(place, "place", torch.int32)
-    _req(weights, "weights", torch.float32, 2)
+    if weights is not None:
+        _req(weights, "weights", torch.float32, 2)
+        top = weights.shape[1]
     _req(out, "out", ndim=2)
-    n, top = weights.shape
-    width = out.shape[1]
-    if y.shape != (n * top, width) or out.shape[0] != n or place.numel() != n * top:
+    n, width = out.shape
+    parts = stride = 0
+    if add is not None:
+        _req(add, "add")
+        if add.dim() not in (2, 3) or tuple(add.shape[-2:]) != (n, width):
+            raise KernelError(f"moe_combine: an output to add of shape {tuple(add.shape)} for {(n, width)}")
+        parts, stride = (add.shape[0], n * width) if add.dim() == 3 else (1, 0)
+    if not top or y.shape != (n * top, width) or (weights is not None and weights.shape[0] != n) or place.numel() != n * top:
         raise KernelError("moe_combine: shapes do not agree")
     if shared is not None:
         _req(shared, "shared", y.dtype, 2)
         if shared.shape != out.shape:
             raise KernelError("moe_combine: the shared output does not fit")
-    _call("gemm", "moe_combine", library().qi_moe_combine, _ptr(y), _code(y), _ptr(place), _ptr(weights), _ptr(shared), _ptr(out),
-          _code(out), n, top, width, _stream())
+    _call("gemm", "moe_combine", library().qi_moe_combine, _ptr(y), _code(y), _ptr(place), _ptr(weights), _ptr(shared), _ptr(add),
+          _code(add) if add is not None else F32, parts, C.c_longlong(stride), _ptr(out), _code(out), n, top, width, _stream())
 
 
 class _LeadRows:
@@ -1690,7 +1755,7 @@ def gated_attention_mma_supported(nq: int, nkv: int, d: int, dv: int) -> bool:
 
 def gated_attention(q, out, k_pages, v_pages, block_table, batch, nq, nkv, d, dv, scale: float, window: int, chunk: int, gate,
                     status, impl: str | None = None, softcap: float = 0.0, out_scale: float = 1.0, sink=None,
-                    key_ranges: int | None = None, bias=None, grouped_heads: bool | None = None) -> None:
+                    key_ranges: int | None = None, bias=None, grouped_heads: bool | None = None, keep_first: int = 0) -> None:
     """Attention with separate key and value sizes, an optional chunk bound and an optional output gate, by the
     kernel that fits: "mma" (bfloat16, head sizes that are multiples of 8 up to 128: flash form on the tensor
     cores, tiles found on the device from the step's arrays) or "generic" (32-bit arithmetic, any sizes). A step
@@ -1702,7 +1767,8 @@ def gated_attention(q, out, k_pages, v_pages, block_table, batch, nq, nkv, d, dv
     "mma" cuts every token's keys into `key_ranges` ranges over separate CTAs (None: as many as fill the device, from
     the longest context and the window, so that a captured step serves its whole context bucket) and adds the parts
     in a second kernel; there the query heads that share a key head are the rows of one tile where there are at most 16
-    of them (`grouped_heads` forces either form). `out` may be a block of columns of wider rows."""
+    of them (`grouped_heads` forces either form). `out` may be a block of columns of wider rows. `keep_first`: the sequence's
+    first keys that stay visible behind a window or a chunk (all three kernels)."""
     if impl is None and q.dtype == torch.bfloat16 and d == dv and not batch.all_decode and batch.tile_req.numel() and (
             gate is None or (gate.stride(0) % 8 == 0 and gate.data_ptr() % 16 == 0)) and attention_prefill_tcgen05_supported(
             nq, nkv, d, k_pages.shape[2], block_table.shape[1]):
@@ -1712,17 +1778,19 @@ def gated_attention(q, out, k_pages, v_pages, block_table, batch, nq, nkv, d, dv
         if lead:
             gated_attention(q[:lead], out[:lead], k_pages, v_pages, block_table[:lead], _LeadRows(batch, lead), nq, nkv, d, dv,
                             scale, window, chunk, gate[:lead] if gate is not None else None, status, impl="mma", softcap=softcap,
-                            out_scale=out_scale, sink=sink, bias=bias)
+                            out_scale=out_scale, sink=sink, bias=bias, keep_first=keep_first)
         return attention_prefill(q, out, k_pages, v_pages, block_table, batch.q_start, batch.start_pos, batch.tile_req,
-                                 batch.tile_q0, nq, nkv, d, scale, window, status, impl="tcgen05", max_kv_len=batch.max_kv_len,
+                                 batch.tile_q0, nq, nkv, d, scale, window, status, impl="tcgen05",
+                                 max_kv_len=min(batch.max_kv_len, window + QUERY_TILE + keep_first) if window else batch.max_kv_len,
                                  key_ranges=1 if chunk else None, chunk=chunk, gate=gate, softcap=softcap, out_scale=out_scale,
-                                 sink=sink, bias=bias)
+                                 sink=sink, bias=bias, keep_first=keep_first)
     if impl is None:
         impl = "mma" if q.dtype == torch.bfloat16 and gated_attention_mma_supported(nq, nkv, d, dv) and (
             gate is None or gate.stride(0) % 2 == 0) else "generic"
     if impl == "generic":
         return attention_generic(q, out, k_pages, v_pages, block_table, batch.positions, batch.token_req, nq, nkv, d, scale,
-                                 window, status, chunk=chunk, gate=gate, softcap=softcap, out_scale=out_scale, sink=sink, bias=bias)
+                                 window, status, chunk=chunk, gate=gate, softcap=softcap, out_scale=out_scale, sink=sink, bias=bias,
+                                 keep_first=keep_first)
     _req_bias(bias, nq)
     if sink is not None:
         _req(sink, "sink", torch.float32, 1)
@@ -1746,7 +1814,7 @@ def gated_attention(q, out, k_pages, v_pages, block_table, batch, nq, nkv, d, dv
     ranges, ws, grouped = 1, None, False
     if getattr(batch, "all_decode", False) and n <= 65535:
         grouped = (nq // nkv <= 16) if grouped_heads is None else grouped_heads
-        keys = min(window or batch.max_kv_len, chunk or batch.max_kv_len, batch.max_kv_len)
+        keys = min(min(window or batch.max_kv_len, chunk or batch.max_kv_len) + keep_first, batch.max_kv_len)
         ranges = key_ranges or max(1, min(-(-keys // 128), 296 // max(n * (nkv if grouped else nq), 1), 64))
         if ranges > 1:
             ws = torch.empty(n * nq * ranges * (dv + 2), dtype=torch.float32, device=q.device)
@@ -1755,4 +1823,4 @@ def gated_attention(q, out, k_pages, v_pages, block_table, batch, nq, nkv, d, dv
           batch.n_requests, n, nq, nkv, d, dv, C.c_float(scale), C.c_float(softcap or 0.0), C.c_float(out_scale), int(window or 0),
           int(chunk or 0), _ptr(gate), C.c_longlong(ldg), _ptr(sink),
           _ptr(bias), bias.shape[1] if bias is not None else 0, ranges, _ptr(ws),
-          int(grouped), C.c_longlong(ldo), _ptr(status), _stream())
+          int(grouped), C.c_longlong(ldo), int(keep_first or 0), _ptr(status), _stream())

@@ -194,6 +194,56 @@ class ParallelGatedBlock(Part):
         return resid, out
 
 
+class ParallelBlock(Part):
+    """One norm, two sublayers side by side on its output:
+
+        h = norm(x) ; x = x + (mixer(h) + ffn(h))
+
+    The two outputs are added in 32-bit before they join the stream: by the feed-forward itself when it offers `forward_add`
+    (a mixture adds the mixer's output, partial sums included, in the kernel that gathers its experts' outputs), else by one
+    kernel. The feed-forward may be absent."""
+
+    def __init__(self, spec, runtime):
+        super().__init__(spec, runtime)
+        if spec.conv is not None or spec.gate_names is not None:
+            raise ConfigError("parallel: this block has neither gates nor input filters (parallel_gated has)")
+        self.norm = build_part("norm", spec.norm, runtime)
+        self.mixer = build_part("mixer", spec.mixer, runtime)
+        self.ffn = build_part("ffn", spec.ffn, runtime) if spec.ffn is not None else None
+        if hasattr(self.mixer, "keep_partials"):
+            self.mixer.keep_partials = True       # what adds the outputs adds a split product's partial sums too
+        self._parts = tuple(p for p in (self.norm, self.mixer, self.ffn) if p is not None)
+
+    @classmethod
+    def needs_of_spec(cls, spec):
+        needs = {}
+        for cat, sub in (("norm", spec.norm), ("mixer", spec.mixer), ("ffn", spec.ffn)):
+            if sub is not None:
+                needs.update(part_class(cat, sub).needs_of_spec(sub))
+        return needs
+
+    def load(self, tensors):
+        for p in self._parts:
+            p.load(tensors)
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def mixer_state_need(self):
+        return getattr(self.mixer, "state_need", lambda: None)()
+
+    def forward(self, resid, delta, batch, cache):
+        h = self.norm(resid, delta)
+        y = self.mixer.forward(h, batch, cache)
+        if self.ffn is None:
+            return resid, y
+        if hasattr(self.ffn, "forward_add"):
+            return resid, self.ffn.forward_add(h, y)
+        out = torch.empty(resid.shape, dtype=torch.float32, device=resid.device)
+        kernels.scaled_sum(y, self.ffn.forward(h), 1.0, 1.0, out)
+        return resid, out
+
+
 class SandwichBlock(Part):
     """A norm before AND after each sublayer, and a multiplier on what joins the stream:
 
@@ -378,3 +428,4 @@ register_part("block", "prenorm", PreNormBlock)
 register_part("block", "sandwich", SandwichBlock)
 register_part("block", "prenorm_conv", ConvPreNormBlock)
 register_part("block", "parallel_gated", ParallelGatedBlock)
+register_part("block", "parallel", ParallelBlock)

@@ -11,7 +11,9 @@ Biases, the gate, the convolution, the cap and the factor are each optional (fie
 softmax's denominator holds exp(b_h) once more, b zero or the learned tensor `sink`); one RMS norm over the whole of q
 and one over the whole of k before the rotation (`q.norm`, `k.norm`); values that are the keys as projected, before
 norm and rotation (no `v` then); or an RMS norm over every head of q and k by itself; a factor on q that grows with the
-position (`q_temp`); a learned number per head that a key's distance adds to its score (`distance_bias`, table `rel`,
+position (`q_temp`); values mixed with those of an earlier layer for the same token (`value_mix`: the layer named "first"
+leaves its values, as projected, with the step; a layer named "mix" caches (1 - a) v + a v_first, a the tensor `vmix`); a
+learned number per head that a key's distance adds to its score (`distance_bias`, table `rel`,
 spread at load to one number a head and distance up to the first distance that reads the last row). The convolution's
 last taps - 1 projected rows are the mixer's state of fixed size BESIDE its pages (`state_need`, handed back as
 `cache.mixer_state`).
@@ -19,7 +21,7 @@ last taps - 1 projected rows are the mixer's state of fixed size BESIDE its page
 Visible keys of the query at position i: j <= i, within the last `window` positions if the spec has a window, and
 within i's own chunk (floor(i / chunk) = floor(j / chunk), chunks counted from the sequence's first position, not
 from where a step began) if it has chunks. The cache need carries both, so pages of chunks a request has left go
-back to the pool at once.
+back to the pool at once. The sequence's first `keep_first` keys stay visible behind both bounds, and their pages stay.
 
 The biases of q, k and v are added where the projection's row is read next (the rotation and cache-write kernel);
 the gate is applied where the attention's result is written; the output projection's bias is left unapplied and
@@ -37,7 +39,9 @@ from ..errors import ConfigError
 from ..weights.loader import TensorNeed
 from .base import Part, register_part
 from .linear import Linear
-from .position import distance_buckets
+from .position import direct_frequencies, distance_buckets
+
+FIRST_VALUES = "first_values"      # the step's key (`batch.extra`) of the values that later layers mix in
 
 
 class GatedAttention(Part):
@@ -58,6 +62,9 @@ class GatedAttention(Part):
             raise ConfigError(f"gated_attention: sink {self.sink_kind!r} / qk_norm {self.qk_norm!r} are not known")
         self.sink = self.q_gain = self.k_gain = self.dist_bias = None
         self.q_temp, self.reach = getattr(s, "q_temp", None), getattr(s, "distance_bias", None)
+        self.keep_first, self.value_mix, self.v_share = int(getattr(s, "keep_first", 0)), getattr(s, "value_mix", None), 0.0
+        if self.keep_first < 0 or self.value_mix not in (None, "first", "mix") or (self.value_mix is not None and self.v_from_k):
+            raise ConfigError(f"gated_attention: keep_first {self.keep_first} / value_mix {self.value_mix!r} cannot be")
         if self.q_temp is not None and self.q_temp[1] < 1:
             raise ConfigError("gated_attention: the query's factor grows every 1 or more positions")
         self.qkv_cols = (self.H + self.G) * self.d + (0 if self.v_from_k else self.G * self.dv)
@@ -75,8 +82,10 @@ class GatedAttention(Part):
         if pos is not None:
             if pos.pairing not in ("half_split", "interleaved") or pos.rotary_dim % 2 or not 0 < pos.rotary_dim <= s.head_dim:
                 raise ConfigError(f"gated_attention: a rotation over {pos.rotary_dim} of {s.head_dim} coordinates ({pos.pairing})")
-            exponent = (2.0 * torch.arange(self.rot // 2, dtype=torch.float64)) / float(self.rot)
-            self.inv_freq = torch.pow(torch.tensor(float(pos.theta), dtype=torch.float64), -exponent).to(torch.float32).to(runtime.device)
+            freqs, magnitude = direct_frequencies(pos)
+            if magnitude != 1.0:
+                raise ConfigError("gated_attention: a rotation that enlarges what it turns is not known here")
+            self.inv_freq = freqs.to(runtime.device)
 
     @classmethod
     def needs_of_spec(cls, s):
@@ -90,6 +99,8 @@ class GatedAttention(Part):
             needs.update({p + "q.norm": TensorNeed((d,), "gain", "gain"), p + "k.norm": TensorNeed((d,), "gain", "gain")})
         if getattr(s, "distance_bias", None) is not None:
             needs[p + "rel"] = TensorNeed((None, H), "gain", "normal")
+        if getattr(s, "value_mix", None) is not None:
+            needs[p + "vmix"] = TensorNeed((), "gain", "half")
         if getattr(s, "sink", None) == "learned":
             needs[p + "sink"] = TensorNeed((H,), "gain", "normal")
         if s.out_gate:
@@ -112,6 +123,8 @@ class GatedAttention(Part):
             rel = tensors[p + "rel"].to(torch.float32)
             buckets = distance_buckets(rel.shape[0], self.reach)
             self.dist_bias = self._gain(rel[torch.tensor(buckets)].t())       # [heads, reach of the last row's edge + 1]
+        if self.value_mix == "mix":
+            self.v_share = float(tensors[p + "vmix"])
         if self.sink_kind == "learned":
             self.sink = self._gain(tensors[p + "sink"])
         if len({t.dtype for t in ws}) > 1:
@@ -126,7 +139,8 @@ class GatedAttention(Part):
             self.out_bias = self._gain(tensors[p + "o.b"])
 
     def cache_need(self):
-        return PagedKVNeed(self.G, self.d, self.spec.window, self.dv if self.dv != self.d else None, self.spec.chunk)
+        return PagedKVNeed(self.G, self.d, self.spec.window, self.dv if self.dv != self.d else None, self.spec.chunk,
+                           self.keep_first if self.spec.window or self.spec.chunk else 0)
 
     def state_need(self):
         """The convolution's state: the last taps - 1 rows of q | k | v as projected (32-bit), beside the pages."""
@@ -152,16 +166,23 @@ class GatedAttention(Part):
             gate_src, proj = proj, conved
         else:
             gate_src = proj
+        v_first = None
+        if self.value_mix == "first":       # (the projection's own columns: nothing is copied)
+            batch.extra[FIRST_VALUES] = proj[:, (self.H + self.G) * self.d:self.qkv_cols]
+        elif self.value_mix == "mix":
+            v_first = batch.extra[FIRST_VALUES]
         q = torch.empty((n, self.H * self.d), dtype=proj.dtype, device=proj.device)
         kernels.bias_rope_kv(proj, self.bias, q, self.inv_freq, self.rot, self.interleaved, batch.positions, batch.token_req,
                              table, cache.page_size, cache.k_pages if cache.writes else None,
                              cache.v_pages if cache.writes else None, self.H, self.G, self.d, self.dv, rt.status,
                              q_gain=self.q_gain, k_gain=self.k_gain, norm_eps=getattr(s, "qk_norm_eps", 0.0),
-                             values_from_keys=self.v_from_k, head_norm=self.qk_norm == "head", q_temp=self.q_temp)
+                             values_from_keys=self.v_from_k, head_norm=self.qk_norm == "head", q_temp=self.q_temp,
+                             v_first=v_first, v_share=self.v_share)
         gate = gate_src[:, self.qkv_cols:self.qkv_cols + self.H * self.dv] if s.out_gate else None
         kernels.gated_attention(q, out, cache.k_pages, cache.v_pages, table, batch, self.H, self.G, self.d, self.dv, s.scale,
                                 s.window or 0, s.chunk or 0, gate, rt.status, softcap=getattr(s, "softcap", None) or 0.0,
-                                out_scale=out_scale * getattr(s, "out_scale", 1.0), sink=self.sink, bias=self.dist_bias)
+                                out_scale=out_scale * getattr(s, "out_scale", 1.0), sink=self.sink, bias=self.dist_bias,
+                                keep_first=self.keep_first)
 
 
 register_part("mixer", "gated_attention", GatedAttention)

@@ -16,6 +16,9 @@ kv_rank + rot_dim, "value" the row's first kv_rank numbers), and the result is t
 Wuv_h. The projections of q and of the latent are one product over the stacked weights. A layer that shares
 another layer's latent has no Wdkv and reads that layer's cache entry with its own Wuk, Wuv, window and sinks.
 
+With `q_rank` in the spec the queries come through a latent of their own, q = Wuq rmsnorm(Wdq x): Wdq and Wdkv are then the
+stacked product, one kernel normalises both latents and writes the cache row, and Wuq is a second product.
+
 Every size and constant is a field of the spec. The angles of the rotation are computed in the kernel from
 32-bit frequencies, theta^(-2i / rotary_dim), so there is no table and no limit on positions. The pairs are
 neighbours (2i, 2i + 1) or halves (i, i + rotary_dim / 2), as the position spec says; its `stretch` (frequencies of
@@ -49,15 +52,19 @@ class LatentAttention(Part):
         self.q_width = self.H * (self.d + self.r)
         self.out_gate = bool(getattr(s, "out_gate", False))
         self.kv_width = 0 if s.shares_latent else self.R + self.r
-        n_out = self.q_width + self.kv_width + (self.H * self.e if self.out_gate else 0)
+        self.q_rank = getattr(s, "q_rank", None)
+        if self.q_rank is not None and (s.shares_latent or self.out_gate):
+            raise ConfigError("latent_attention: a query latent comes without a shared latent and without an output gate")
+        self.uq = Linear(runtime, self.q_width, self.q_rank, s.prefix + "uq") if self.q_rank else None
+        n_out = (self.q_rank or self.q_width) + self.kv_width + (self.H * self.e if self.out_gate else 0)
         self.proj = Linear(runtime, n_out, s.hidden_size, s.prefix + "q+dkv+g")
         self.o = Linear(runtime, s.hidden_size, self.H * self.e, s.prefix + "o")
-        self.uk_t = self.uv = self.gain = self.sink = self.inv_freq = None
+        self.uk_t = self.uv = self.gain = self.q_gain = self.sink = self.inv_freq = None
         self.keep_partials = False      # a block whose next norm adds a split product's partial sums itself sets this
         self.half_split = pos is not None and pos.pairing == "half_split"
         self.magnitude = 1.0
         if self.rot_dims:
-            if getattr(pos, "stretch", None) is None and not self.half_split:
+            if getattr(pos, "stretch", None) is None and getattr(pos, "bands", None) is None and not self.half_split:
                 # theta^(-2i / dims), exponent and power in 32-bit
                 exponent = (2.0 * torch.arange(self.rot_dims // 2, dtype=torch.float32)) / torch.tensor(float(self.rot_dims), dtype=torch.float32)
                 self.inv_freq = torch.pow(torch.tensor(float(pos.theta), dtype=torch.float32), -exponent).to(runtime.device)
@@ -68,7 +75,12 @@ class LatentAttention(Part):
     @classmethod
     def needs_of_spec(cls, s):
         p, H = s.prefix, s.num_heads
-        needs = {p + "q": TensorNeed((H * (s.head_dim + s.rot_dim), s.hidden_size))}
+        Q = getattr(s, "q_rank", None)
+        if Q is not None:
+            needs = {p + "dq": TensorNeed((Q, s.hidden_size)), p + "dq.norm": TensorNeed((Q,), "gain", "gain"),
+                     p + "uq": TensorNeed((H * (s.head_dim + s.rot_dim), Q))}
+        else:
+            needs = {p + "q": TensorNeed((H * (s.head_dim + s.rot_dim), s.hidden_size))}
         if not s.shares_latent:
             needs[p + "dkv"] = TensorNeed((s.kv_rank + s.rot_dim, s.hidden_size))
             needs[p + "dkv.norm"] = TensorNeed((s.kv_rank,), "gain", "gain")
@@ -83,11 +95,14 @@ class LatentAttention(Part):
 
     def load(self, tensors):
         s, p, rt = self.spec, self.spec.prefix, self.runtime
-        stack = [tensors[p + "q"]] + ([] if s.shares_latent else [tensors[p + "dkv"]]) + ([tensors[p + "g"]] if self.out_gate else [])
+        stack = [tensors[p + ("dq" if self.q_rank else "q")]] + ([] if s.shares_latent else [tensors[p + "dkv"]]) + ([tensors[p + "g"]] if self.out_gate else [])
         if len({t.dtype for t in stack}) > 1:
             stack = [t.to(torch.float32) for t in stack]
         self.proj.load(torch.cat(stack, dim=0))
         self.o.load(tensors[p + "o"])
+        if self.q_rank:
+            self.uq.load(tensors[p + "uq"])
+            self.q_gain = self._gain(tensors[p + "dq.norm"])
         wdt = torch.float32 if rt.dtype == torch.float32 else None
         uk = tensors[p + "uk"].reshape(self.H, self.d, self.R)
         # into the latent space: ql_h = Wuk_h^T q_h, as a product with weight [R, d] per head
@@ -108,8 +123,17 @@ class LatentAttention(Part):
         W = self.R + self.r
         table = batch.block_tables[cache.group]
         writes = cache.writes and not s.shares_latent
-        z = self.proj(x)                                        # [n, H (d + r) (+ R + r) (+ H e)]
         q = torch.empty((n, self.H, W), dtype=x.dtype, device=x.device)
+        if self.q_rank:
+            if not cache.writes:
+                raise ConfigError("latent_attention: a layer with a query latent writes its own cache entry")
+            cq = torch.empty((n, self.q_rank), dtype=x.dtype, device=x.device)
+            kernels.latent_down(self.proj(x, keep_partials=True), self.q_rank, self.q_gain, cq, self.gain, s.norm_eps, self.inv_freq, self.rot_dims,
+                                batch.positions, batch.token_req, table, cache.k_pages, self.r, self.R, rt.status,
+                                half_split=self.half_split, magnitude=self.magnitude)
+            z, writes = self.uq(cq), False                      # [n, H (d + r)]; the cache row is written
+        else:
+            z = self.proj(x)                                    # [n, H (d + r) (+ R + r) (+ H e)]
         kernels.latent_prepare(z, self.q_width if writes else None, q, self.gain, s.norm_eps, self.inv_freq, self.rot_dims,
                                batch.positions, batch.token_req, table, cache.k_pages, self.H, self.d, self.r, self.R, rt.status,
                                half_split=self.half_split, magnitude=self.magnitude)

@@ -1,13 +1,19 @@
-"""Feed-forwards of the clamped gated form, alone and as a routed mixture.
+"""Feed-forwards of the clamped gated form, and routed mixtures of small feed-forwards.
 
-    expert(x) = down(g * sigmoid(alpha g) * (u + 1)),   g = min(gate(x), limit),  u = clamp(up(x), -limit, limit)
+    clamped(x) = down(g * sigmoid(alpha g) * (u + 1)),   g = min(gate(x), limit),  u = clamp(up(x), -limit, limit)
+    gated(x)   = down(silu(gate(x)) * up(x))
 
-`ClampedGLU` is one such feed-forward for every token (gate and up stacked into one product). `MoE` routes:
+`ClampedGLU` is one clamped feed-forward for every token (gate and up stacked into one product). `MoE` routes between
+experts of either form:
 
-    s       = softmax(router(x))                        over all experts, 32-bit
-    chosen  = the `top` largest of s + correction       (the correction steers the choice only)
-    w_k     = s_k / (sum of the chosen s + 1e-20) * router_scale
-    y       = sum_k w_k expert_k(x)  (+ shared(x))
+    s       = softmax(router(x)) over all experts, or sigmoid(router(x)); 32-bit
+    chosen  = the `top` largest of s + correction       (the optional correction steers the choice only)
+    w_k     = s_k / (sum of the chosen s + 1e-20) * router_scale, or s_k * router_scale as they are
+    y       = sum_k w_k expert_k(x)  (+ shared(x)),   or   sum_k expert_k(w_k x)   with the weight on the input
+
+A weight on a gated expert's input is applied to what gate and up make of it, which are linear in it: w gate(x) and
+w up(x), in 32-bit, in the product's epilogue with the activation (a step that runs expert by expert scales the rows as it
+gathers them).
 
 The tokens are grouped by expert on the device: the (token, choice) pairs are sorted by expert, each expert's rows
 form tiles of their own, and ONE grouped launch per projection runs every expert over exactly its rows; no count
@@ -24,6 +30,7 @@ from __future__ import annotations
 import torch
 
 from .. import kernels
+from ..config.spec import ClampedGLUSpec
 from ..errors import ConfigError
 from ..weights.loader import TensorNeed
 from .base import Part, register_part
@@ -63,6 +70,13 @@ class MoE(Part):
         s = spec
         if not 0 < s.top <= s.experts:
             raise ConfigError(f"moe: {s.top} of {s.experts} experts a token")
+        if s.scoring not in ("softmax", "sigmoid") or s.weight_on not in ("output", "input"):
+            raise ConfigError(f"moe: scores {s.scoring!r} / weights on {s.weight_on!r} are not known")
+        self.clamped = isinstance(s.expert, ClampedGLUSpec)
+        if not self.clamped and s.expert.activation != "silu":
+            raise ConfigError(f"moe: experts with {s.expert.activation!r} have no kernel (silu, or the clamped form)")
+        if self.clamped and s.weight_on == "input":
+            raise ConfigError("moe: a weight on the input of a clamped expert has no kernel")
         self.router = Linear(runtime, s.experts, s.hidden_size, s.prefix + "router")
         self.shared = ClampedGLU(s.shared, runtime) if s.shared is not None else None
         self.w_gate_up = self.w_down = self.correction = None
@@ -74,7 +88,8 @@ class MoE(Part):
         for e in range(s.experts):
             needs.update({f"{p}e{e}.gate": TensorNeed((i, h)), f"{p}e{e}.up": TensorNeed((i, h)), f"{p}e{e}.down": TensorNeed((h, i))})
         needs[p + "router"] = TensorNeed((s.experts, h))
-        needs[p + "correction"] = TensorNeed((s.experts,), "matrix", "zeros")
+        if s.has_correction:
+            needs[p + "correction"] = TensorNeed((s.experts,), "matrix", "zeros")
         if s.shared is not None:
             needs.update(ClampedGLU.needs_of_spec(s.shared))
         return needs
@@ -82,8 +97,13 @@ class MoE(Part):
     def load(self, tensors):
         s, p, rt = self.spec, self.spec.prefix, self.runtime
         self.router.load(tensors[p + "router"])
-        self.correction = self._gain(tensors[p + "correction"])
-        gu = torch.stack([torch.cat([tensors[f"{p}e{e}.gate"], tensors[f"{p}e{e}.up"]], dim=0) for e in range(s.experts)])
+        if s.has_correction:
+            self.correction = self._gain(tensors[p + "correction"])
+        pairs = [(tensors[f"{p}e{e}.gate"], tensors[f"{p}e{e}.up"]) for e in range(s.experts)]
+        if self.clamped:
+            gu = torch.stack([torch.cat(gu, dim=0) for gu in pairs])
+        else:       # rows in (gate, up) pairs: the activation rides in the product's epilogue
+            gu = torch.stack([torch.stack(gu, dim=1).flatten(0, 1) for gu in pairs])
         down = torch.stack([tensors[f"{p}e{e}.down"] for e in range(s.experts)])
         if rt.dtype == torch.float32:
             gu, down = gu.to(torch.float32), down.to(torch.float32)
@@ -100,35 +120,51 @@ class MoE(Part):
                 and not torch.cuda.is_current_stream_capturing())
 
     def forward(self, x):
+        return self._run(x, None, x.dtype)
+
+    def forward_add(self, x, other):
+        """The mixture's output plus `other` (the same tokens' output of a sublayer side by side with this one, whole or as
+        partial sums), in 32-bit: added by the kernel that gathers the experts' outputs."""
+        return self._run(x, other, torch.float32)
+
+    def _run(self, x, other, out_dtype):
         s = self.spec
         n, dev = x.shape[0], x.device
         pairs, ff = n * s.top, s.expert.intermediate_size
         logits = self.router(x, out_dtype=torch.float32)
         ids = torch.empty((n, s.top), dtype=torch.int32, device=dev)
         weights = torch.empty((n, s.top), dtype=torch.float32, device=dev)
-        kernels.moe_route(logits, self.correction, ids, weights, s.router_scale)
+        kernels.moe_route(logits, self.correction, ids, weights, s.router_scale, s.scoring, s.normalize)
         offsets = torch.empty(s.experts + 1, dtype=torch.int32, device=dev)
         order = torch.empty(pairs, dtype=torch.int32, device=dev)
         place = torch.empty(pairs, dtype=torch.int32, device=dev)
         tiles = torch.empty((min(pairs, pairs // kernels.moe_tile_rows() + s.experts), 3), dtype=torch.int32, device=dev)
         kernels.moe_group(ids, s.experts, offsets, order, place, tiles)
-        gu = torch.empty((pairs, 2 * ff), dtype=x.dtype, device=dev)
         a = torch.empty((pairs, ff), dtype=x.dtype, device=dev)
         y = torch.empty((pairs, s.hidden_size), dtype=x.dtype, device=dev)
+        on_input = weights if s.weight_on == "input" else None
         if self._by_expert(x, pairs):
             bounds = offsets.tolist()          # the one place where such a step waits for the device
             xs = torch.empty((pairs, s.hidden_size), dtype=x.dtype, device=dev)
-            kernels.moe_gather(x, order, s.top, xs)
-            kernels.moe_gemm_by_expert(xs, self.w_gate_up, gu, bounds, self.runtime.status)
-            kernels.glu_clamped(gu, a, s.expert.limit, s.expert.alpha)
+            kernels.moe_gather(x, order, s.top, xs, pair_scale=on_input)
+            if self.clamped:
+                gu = torch.empty((pairs, 2 * ff), dtype=x.dtype, device=dev)
+                kernels.moe_gemm_by_expert(xs, self.w_gate_up, gu, bounds, self.runtime.status)
+                kernels.glu_clamped(gu, a, s.expert.limit, s.expert.alpha)
+            else:
+                kernels.moe_gemm_by_expert(xs, self.w_gate_up, a, bounds, self.runtime.status, epilogue="silu_mul")
             kernels.moe_gemm_by_expert(a, self.w_down, y, bounds, self.runtime.status)
         else:
-            kernels.moe_gemm(x, self.w_gate_up, gu, tiles, order, s.top, gather=True)
-            kernels.glu_clamped(gu, a, s.expert.limit, s.expert.alpha)
+            if self.clamped:
+                gu = torch.empty((pairs, 2 * ff), dtype=x.dtype, device=dev)
+                kernels.moe_gemm(x, self.w_gate_up, gu, tiles, order, s.top, gather=True)
+                kernels.glu_clamped(gu, a, s.expert.limit, s.expert.alpha)
+            else:
+                kernels.moe_gemm(x, self.w_gate_up, a, tiles, order, s.top, gather=True, epilogue="silu_mul", pair_scale=on_input)
             kernels.moe_gemm(a, self.w_down, y, tiles, order, s.top, gather=False)
         shared = self.shared.forward(x) if self.shared is not None else None
-        out = torch.empty((n, s.hidden_size), dtype=x.dtype, device=dev)
-        kernels.moe_combine(y, place, weights, shared, out)
+        out = torch.empty((n, s.hidden_size), dtype=out_dtype, device=dev)
+        kernels.moe_combine(y, place, weights if on_input is None else None, shared, out, add=other, top=s.top)
         return out
 
     __call__ = forward

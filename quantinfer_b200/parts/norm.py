@@ -112,6 +112,17 @@ class RMSNorm(Part):
     __call__ = forward
 
 
+class NamedRMSNorm(RMSNorm):
+    """RMS norm with a gain per coordinate whose tensor is named by the spec's `prefix` itself."""
+
+    @classmethod
+    def needs_of_spec(cls, spec):
+        return {spec.prefix: TensorNeed((spec.size,), "gain", "gain")}
+
+    def load(self, tensors):
+        self.gain = self._gain(tensors[self.spec.prefix])
+
+
 class OnePlusRMSNorm(RMSNorm):
     """RMS norm whose weight is stored around zero: out = x / sqrt(mean(x^2) + eps) * (1 + w), w the tensor named by the
     spec's `prefix` itself. 1 + w is formed once, in 32-bit, at load. Besides the pre-norm form of every norm it offers
@@ -257,6 +268,7 @@ class StreamSumNorm(Part):
     __call__ = forward
 
 
+register_part("norm", "rmsnorm_named", NamedRMSNorm)
 register_part("norm", "layernorm_nobias", GainLayerNorm)
 register_part("norm", "stream_sum", StreamSumNorm)
 register_part("norm", "rmsnorm", RMSNorm)

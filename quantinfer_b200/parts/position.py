@@ -32,11 +32,23 @@ def direct_frequencies(spec):
     slow): with where(t) = rotary_dim ln(original / (2 pi t)) / (2 ln theta) the pair's number at which a pair turns t
     times over `original` positions, lo = max(floor(where(fast)), 0), hi = min(ceil(where(slow)), rotary_dim - 1) and
     ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), pair i turns by f_i / factor * ramp_i + f_i (1 - ramp_i), and cos
-    and sin are multiplied by 0.1 ln(factor) + 1. Evaluated in 64-bit and rounded once."""
+    and sin are multiplied by 0.1 ln(factor) + 1. With `bands` = (factor, low, high, original): by wavelength l = 2 pi / f_i, f_i
+    below original / high, f_i / factor above original / low, (1 - s) f_i / factor + s f_i between them with s = (original / l -
+    low) / (high - low). Evaluated in 64-bit and rounded once."""
     dims = spec.rotary_dim
     i = torch.arange(dims // 2, dtype=torch.float64)
     f = torch.pow(torch.tensor(float(spec.theta), dtype=torch.float64), -2.0 * i / float(dims))
-    stretch = getattr(spec, "stretch", None)
+    stretch, bands = getattr(spec, "stretch", None), getattr(spec, "bands", None)
+    if stretch is not None and bands is not None:
+        raise ConfigError("a rotation is stretched by one rule at most")
+    if bands is not None:
+        factor, low, high, original = (float(x) for x in bands)
+        if min(factor, low, high, original) <= 0.0 or high < low:
+            raise ConfigError("a rotation in frequency bands needs positive factor, low, high and original, high at least low")
+        length = 2.0 * math.pi / f
+        s = (original / length - low) / max(high - low, 1e-300)
+        mixed = (1.0 - s) * f / factor + s * f
+        f = torch.where(length < original / high, f, torch.where(length > original / low, f / factor, mixed))
     if stretch is None:
         return f.to(torch.float32), 1.0
     factor, original, fast, slow = (float(x) for x in stretch)

@@ -44,7 +44,7 @@ from .safetensors_io import SafeTensorsFolder
 class TensorNeed:
     shape: tuple             # a dimension may be None: any size (the part reads it from the tensor it is given)
     kind: str = "matrix"     # "matrix" | "table" (embedding) | "gain" | "int"
-    init: str = "normal"     # how random weights fill it: "normal" | "gain" | "zeros"
+    init: str = "normal"     # how random weights fill it: "normal" | "gain" | "zeros" | "identity" | "half"
     free: int = 16           # the size a None dimension gets when weights are drawn at random
 
     def fits(self, shape) -> bool:

@@ -37,6 +37,9 @@ def random_tensor(need: TensorNeed, seed: int, index: int, dtype: torch.dtype, d
     if need.init == "identity":             # what mixes residual streams: every stream mostly itself
         u = torch.rand(need.shape, generator=g, dtype=torch.float32, device=device)
         return torch.eye(*need.shape, device=device) + (u * 2.0 - 1.0) * GAIN_SPREAD
+    if need.init == "half":                 # a share between two things
+        u = torch.rand(need.shape, generator=g, dtype=torch.float32, device=device)
+        return 0.5 + (u * 2.0 - 1.0) * GAIN_SPREAD
     if need.init == "zeros":
         return torch.zeros(need.shape, dtype=dtype, device=device)
     t = torch.randn(need.shape, generator=g, dtype=torch.float32, device=device) * MATRIX_STD
