@@ -309,8 +309,46 @@ def siditar_arithmetic(config, spec):
     return a
 
 
+def bomipel_arithmetic(config, spec):
+    """The same for a model of the Bomipel design: per layer the mixer's projections (grouped attention: q, k, v, out; latent
+    attention: both latents, the heads' queries, the per-head products, out), the mixture a token runs (router, `top` experts),
+    attention over the window and the kept first keys, or over every earlier row of the latent. `weight_bytes` counts what a
+    decode step of `batch` tokens reads of a mixture: the experts it can be expected to touch."""
+    from quantinfer_b200.config.bomipel import BomipelAttention
+
+    H, V = spec.hidden_size, spec.vocab_size
+    active = stored = touched = 0
+    batch, groups, latents = COMPARE_BATCH, [], []
+    for layer in config.layers:
+        m, f = layer.mixer, layer.mlp
+        if isinstance(m, BomipelAttention):
+            mix = H * ((m.heads + m.kv_heads) * m.dim + m.kv_heads * m.vdim) + m.heads * m.vdim * H
+            groups.append((m.heads, m.dim, m.vdim, m.kv_heads, (m.window + m.keep_first) if m.window else None))
+        else:
+            mix = H * (m.q_rank + m.kv_rank + m.rot_dim) + m.q_rank * m.heads * (m.dim + m.rot_dim)
+            mix += m.heads * m.kv_rank * (m.dim + m.vdim) + m.heads * m.vdim * H
+            latents.append((m.heads, m.kv_rank, m.rot_dim))
+        active += mix; stored += mix; touched += mix
+        if f is not None:
+            one, router = 3 * H * f.ff, f.experts * H
+            active += f.top * one + router
+            stored += f.experts * one + router
+            touched += f.experts * (1.0 - (1.0 - f.top / f.experts) ** batch) * one + router
+    a = dict(L=len(config.layers), H=H, V=V, layer_params=active / len(config.layers), stored_params=stored)
+    a["weight_bytes"] = 2 * (touched + V * H)
+    a["kv_bytes_per_token"] = 0
+    a["kv_bytes"] = lambda ctx: (sum(2 * g * (d + dv) * (min(ctx, w) if w else ctx) for _, d, dv, g, w in groups)
+                                 + sum(2 * (R + r) * ctx for _, R, r in latents))
+    a["gemm_flops"] = lambda T, rows_=1: 2.0 * T * active + 2.0 * H * V * rows_
+    a["attn_flops"] = lambda T: (sum(2.0 * h * (d + dv) * sum(min(t + 1, w or T) for t in range(T)) for h, d, dv, _, w in groups)
+                                 + sum(2.0 * h * (2 * R + r) * (T * (T + 1) / 2) for h, R, r in latents))
+    return a
+
+
 def model_arithmetic(config, spec):
     """Parameter counts, bytes and flops of the configuration (every matrix bf16)."""
+    if type(config).__name__ == "BomipelConfig":
+        return bomipel_arithmetic(config, spec)
     if type(config).__name__ == "SiditarConfig":
         return siditar_arithmetic(config, spec)
     if type(config).__name__ == "LemotarConfig":
@@ -745,6 +783,52 @@ def compare_siditar(args):
     return compare_kiruvik(args, "Siditar layers beside Dulotar layers of equal width", SIDITAR_SIZES, siditar_entries)
 
 
+# ---- the Bomipel design beside Kiruvik and Bebuvik layers of equal width ------------------------------------------
+# (width, softmax heads / kv heads of 128 behind a window of 1,024 and four kept keys, latent-attention heads of 64 + 64 with
+# values of 128 over a latent of 256 and a query latent, experts x their feed-forward, four of which a token uses): four layers,
+# latent, grouped, grouped (values mixed), latent, each beside its mixture. No other design has all of it: Kiruvik layers
+# (grouped attention in chunks of 1,024 and mixtures of the same experts) are the closest for attention and mixture, Bebuvik
+# layers (latent attention and a dense feed-forward side by side on one norm; the feed-forward holds what a token runs of the
+# mixture) for the latent attention and the block
+BOMIPEL_SIZES = {
+    "2048": dict(width=2048, heads=16, kv=4, rank=256, qrank=768, experts=16, eff=1024),
+    "4096": dict(width=4096, heads=32, kv=8, rank=256, qrank=1536, experts=32, eff=1536),
+}
+BOMIPEL_TOP = 4
+
+
+def bomipel_entries(size):
+    z = BOMIPEL_SIZES[size]
+    att = {"heads": z["heads"], "kv_heads": z["kv"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "v_mix": True,
+           "rot": {"base": 500000.0, "dims": 128, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048}},
+           "mask": {"size": KIRUVIK_CHUNK, "keep_first": 4}}
+    lat = {"heads": z["heads"], "dim": 64, "rot_dim": 64, "vdim": 128, "q_rank": z["qrank"], "kv_rank": z["rank"], "scale": 128 ** -0.5,
+           "rot": {"base": 500000.0, "dims": 64}}
+    mix = {"kind": "moe", "router": {"experts": z["experts"], "top": BOMIPEL_TOP}, "expert": {"ff": z["eff"]}}
+    new = dict(architecture="Bomipel", vocab=COMPARE_VOCAB, width=z["width"], norm={"eps": 1e-6}, logit_softcap=30.0,
+               layers=[{"type": t, "mixer": m, "mlp": mix} for t, m in (("latent_attention", lat), ("attention", att), ("attention", att),
+                                                                        ("latent_attention", lat))])
+    old_att = {"heads": z["heads"], "kv_heads": z["kv"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": {"base": 500000.0, "dims": 64},
+               "mask": {"size": KIRUVIK_CHUNK}}
+    old_mix = {"kind": "moe", "router": {"experts": z["experts"], "top": BOMIPEL_TOP, "scale": 1.0}, "expert": {"ff": z["eff"], "limit": 7.0}}
+    kir = dict(architecture="Kiruvik", vocab=COMPARE_VOCAB, width=z["width"], norm={"eps": 1e-6}, residual_mult=0.6,
+               layers=[{"type": "attention", "mixer": old_att, "mlp": old_mix}] * COMPARE_LAYERS)
+    old_lat = {"heads": z["heads"], "dim": 64, "rot_dim": 64, "vdim": 128, "kv_rank": z["rank"], "scale": 128 ** -0.5,
+               "rot": {"base": 500000.0, "dims": 64}}
+    beb = dict(architecture="Bebuvik", vocab=COMPARE_VOCAB, width=z["width"], norm={"eps": 1e-6}, canon={"taps": 4},
+               embedding={"bigram": {"buckets": 65521, "mul_prev": 8191, "mul_cur": 31}}, logit_softcap=30.0,
+               layers=[{"type": "latent_attention", "mixer": old_lat, "mlp": {"kind": "dense", "ff": 3 * BOMIPEL_TOP * z["eff"] // 2}}] * COMPARE_LAYERS)
+    common = dict(seed=5, prompt_len=COMPARE_PROMPT, context=4096, batch=COMPARE_BATCH, points=())
+    return tuple(dict(common, config=c, name=f"{c['architecture']} layers of width {size}") for c in (new, kir, beb))
+
+
+def compare_bomipel(args):
+    """Prefill and decode throughput of four Bomipel layers (latent attention and windowed grouped attention, each beside a
+    mixture of gated experts) beside four Kiruvik layers (grouped attention and mixtures of the same experts) and four Bebuvik
+    layers (latent attention) of the same width, and each kernel class of all alone with its share of the roofline."""
+    return compare_kiruvik(args, "Bomipel layers beside Kiruvik and Bebuvik layers of equal width", BOMIPEL_SIZES, bomipel_entries)
+
+
 def compare_kiruvik(args, title="Kiruvik layers beside dense GQA (Qwen3) layers of equal width", sizes=None, entries_of=None):
     """Prefill and decode throughput of four Kiruvik layers (attention and state-space mixers, dense and routed
     feed-forwards) beside four dense GQA layers of the same width, heads and vocabulary, and each kernel class of both
@@ -1080,7 +1164,7 @@ def main() -> int:
                     help="run one part only (for profiler captures of a small case)")
     ap.add_argument("--timeline", action="store_true",
                     help="build the kernels with their time stamps and print where a decode step's time goes, kernel by kernel")
-    ap.add_argument("--compare", nargs="?", const="bebuvik", default=None, choices=["bebuvik", "kiruvik", "dulotar", "lemotar", "siditar"],
+    ap.add_argument("--compare", nargs="?", const="bebuvik", default=None, choices=["bebuvik", "kiruvik", "dulotar", "lemotar", "siditar", "bomipel"],
                     help="instead of the headline workload: layers of another design (default: the latent-attention design) "
                          "beside dense GQA layers of equal sizes")
     ap.add_argument("--compare-sizes", default=None, help="widths to compare, with commas between them (default: all)")
@@ -1109,7 +1193,8 @@ def main() -> int:
     torch.cuda.set_device(0)
     if args.compare:
         args.skip_points = args.skip_classes = True
-        run = {"kiruvik": compare_kiruvik, "dulotar": compare_dulotar, "bebuvik": compare_designs, "lemotar": compare_lemotar, "siditar": compare_siditar}[args.compare]
+        run = {"kiruvik": compare_kiruvik, "dulotar": compare_dulotar, "bebuvik": compare_designs, "lemotar": compare_lemotar, "siditar": compare_siditar,
+               "bomipel": compare_bomipel}[args.compare]
         print(json.dumps(run(args)))
         return 0
     if args.only == "mixed":

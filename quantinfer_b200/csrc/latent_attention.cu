@@ -106,7 +106,7 @@ latent_prepare_kernel(const TP* __restrict__ proj, long long ldp, int kv_off, T*
 }
 
 template <typename TP, typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(512)
 latent_down_kernel(const TP* __restrict__ proj, int parts, size_t part_stride, long long ldp, int Q, const float* __restrict__ q_gain,
                    T* __restrict__ cq, const float* __restrict__ gain, float eps, const float* __restrict__ inv_freq, int rot_dims,
                    const int* __restrict__ positions, const int* __restrict__ token_req, const int* __restrict__ block_table,
@@ -121,7 +121,7 @@ latent_down_kernel(const TP* __restrict__ proj, int parts, size_t part_stride, l
     float sq = 0.f, sc = 0.f;
     for (int i = threadIdx.x; i < total; i += blockDim.x) {
         float v = qi::to_f32<TP>(src[i]);
-#pragma unroll 4
+#pragma unroll 8
         for (int k = 1; k < parts; ++k) v += qi::to_f32<TP>(src[k * part_stride + i]);
         row[i] = v;
         if (i < Q) sq = fmaf(v, v, sq);
@@ -305,9 +305,10 @@ extern "C" int qi_latent_down(const void* proj, int proj_dtype, int parts, long 
     const size_t smem = sizeof(float) * (size_t)(Q + R + r);
     QI_REQUIRE(smem <= 47 * 1024, "latent_down: a row of %d + %d + %d is too wide for this kernel", Q, R, r);
     if (n_tokens == 0) return 0;
+    const int threads = n_tokens <= 296 ? 512 : 128;      // few tokens: more of a row's loads in flight
     QI_DISPATCH_DTYPE(proj_dtype, TP, {
         QI_DISPATCH_DTYPE(dtype, T, {
-            qi::launch(latent_down_kernel<TP, T>, dim3(n_tokens), dim3(128), smem, stream, (const TP*)proj, parts, (size_t)part_stride, ldp,
+            qi::launch(latent_down_kernel<TP, T>, dim3(n_tokens), dim3(threads), smem, stream, (const TP*)proj, parts, (size_t)part_stride, ldp,
                        Q, q_gain, (T*)cq, gain, eps, inv_freq, rot_dims, positions, token_req, block_table, max_blocks, page_size,
                        num_pages, (T*)cache, r, R, half_split, magnitude, status);
         });

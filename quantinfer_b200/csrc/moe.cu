@@ -16,6 +16,7 @@
 //   moe_combine   out[t] = sum_k weight[t, k] * y[place of (t, k)] (+ shared[t]) (+ another branch's output, which
 //                 may still be partial sums), k ascending, 32-bit; without weights the plain sum.
 #include "common.cuh"
+#include "attention_frag.cuh"
 #include "vec8.cuh"
 
 #include <math.h>
@@ -219,83 +220,79 @@ moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TY* __restri
 
 // The same product on the tensor cores for bfloat16 operands and results (mma.sync m16n8k16, 32-bit sums, K a
 // multiple of 8): a CTA of four warps takes one row tile (up to 32 sorted rows of one expert) and 64 output columns;
-// the next 32 of K are requested into registers while the current ones are multiplied.
-constexpr int MN = 64, MK = 32, MPAD = 8;
-
-__device__ __forceinline__ void mma_bf16_16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
+// K advances in steps of 64 through four cp.async buffers, three of them in flight, since with few rows an expert the
+// product is the stream of its weights. Rows are padded by 16 bytes against ldmatrix bank conflicts.
+constexpr int MN = 64, MK = 64, kMoeStages = 4, kMoeStride = MK * 2 + 16;
+constexpr int kMoeStageBytes = (BM + MN) * kMoeStride, kMoeSmem = kMoeStages * kMoeStageBytes;
 
 __global__ void __launch_bounds__(128)
 moe_gemm_mma_kernel(const qi::bf16* __restrict__ x, const qi::bf16* __restrict__ w, qi::bf16* __restrict__ y,
                     const int* __restrict__ tiles, const int* __restrict__ order, int top, int gather, int N, int K,
                     long long ldx, long long ldy, int n_src, int n_rows, int n_experts, int epilogue,
                     const float* __restrict__ pair_scale) {
-    __shared__ __align__(16) qi::bf16 As[BM][MK + MPAD];
-    __shared__ __align__(16) qi::bf16 Bs[MN][MK + MPAD];
-    __shared__ int src_row[BM];
+    extern __shared__ __align__(128) unsigned char moe_smem[];
     qi::pdl_wait();
     const int expert = tiles[3 * blockIdx.y], row0 = tiles[3 * blockIdx.y + 1], rows = tiles[3 * blockIdx.y + 2];
     if (expert < 0 || expert >= n_experts || row0 < 0 || rows < 0 || rows > BM || row0 + rows > n_rows) return;
     const qi::bf16* we = w + (size_t)expert * N * K;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int n0 = blockIdx.x * MN;
-    if (tid < BM) src_row[tid] = tid < rows ? (gather ? order[row0 + tid] / top : row0 + tid) : -1;
-    if (tid < BM && (src_row[tid] < 0 || src_row[tid] >= n_src)) src_row[tid] = -1;
-    __syncthreads();
-    const int ar = tid >> 2, ac = (tid & 3) * 8;           // this thread's 16-byte piece of the A tile (32 x 32)
-    const qi::bf16* a_src = src_row[ar] >= 0 ? x + (size_t)src_row[ar] * ldx + ac : nullptr;
-    const qi::bf16* b_src[2];
+    // this thread's 16-byte pieces of a stage: column piece tid % 8 of rows tid / 8 + 16 i, two of A and four of B
+    const int pr = tid >> 3, pc = (tid & 7) * 8;
+    const qi::bf16* a_src[2];
+    const qi::bf16* b_src[4];
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {                          // and its two pieces of the B tile (64 x 32)
-        const int br = (tid >> 2) + 32 * i;
-        b_src[i] = n0 + br < N ? we + (size_t)(n0 + br) * K + ac : nullptr;
+    for (int i = 0; i < 2; ++i) {
+        const int r = pr + 16 * i;
+        const int src = r < rows ? (gather ? order[row0 + r] / top : row0 + r) : -1;
+        a_src[i] = (src >= 0 && src < n_src) ? x + (size_t)src * ldx + pc : nullptr;
     }
-    auto fetch = [&](int k0, uint4& a, uint4 (&b)[2]) {
-        const bool in = k0 + ac < K;
-        a = (in && a_src) ? *reinterpret_cast<const uint4*>(a_src + k0) : make_uint4(0u, 0u, 0u, 0u);
 #pragma unroll
-        for (int i = 0; i < 2; ++i) b[i] = (in && b_src[i]) ? *reinterpret_cast<const uint4*>(b_src[i] + k0) : make_uint4(0u, 0u, 0u, 0u);
+    for (int i = 0; i < 4; ++i) b_src[i] = n0 + pr + 16 * i < N ? we + (size_t)(n0 + pr + 16 * i) * K + pc : nullptr;
+    const uint32_t base = qi_attn::smem_u32(moe_smem), mine = base + pr * kMoeStride + pc * 2;
+    auto piece = [&](uint32_t dst, const qi::bf16* src, int k0) {
+        const bool real = src && k0 + pc < K;
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(real ? (const void*)(src + k0) : (const void*)w), "r"(real ? 16 : 0) : "memory");
+    };
+    const int steps = (K + MK - 1) / MK;
+    auto request = [&](int it) {
+        if (it < steps) {
+            const uint32_t dst = mine + (it % kMoeStages) * kMoeStageBytes;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) piece(dst + (BM + 16 * i) * kMoeStride, b_src[i], it * MK);
+#pragma unroll
+            for (int i = 0; i < 2; ++i) piece(dst + 16 * i * kMoeStride, a_src[i], it * MK);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");      // (an empty group past the end keeps the count)
     };
     float acc[2][2][4];
 #pragma unroll
     for (int i = 0; i < 2; ++i)
 #pragma unroll
         for (int j = 0; j < 2; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
-    uint4 a_reg, b_reg[2];
-    fetch(0, a_reg, b_reg);
-    for (int k0 = 0; k0 < K; k0 += MK) {
-        __syncthreads();
-        *reinterpret_cast<uint4*>(&As[ar][ac]) = a_reg;
+    const int m_tiles = rows > 16 ? 2 : 1;
+    for (int it = 0; it < kMoeStages - 1; ++it) request(it);
+    for (int it = 0; it < steps; ++it) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(kMoeStages - 2) : "memory");
+        __syncthreads();          // this stage has landed, and every warp has left the one that is requested next
+        request(it + kMoeStages - 1);
+        const uint32_t as = base + (it % kMoeStages) * kMoeStageBytes, bs = as + BM * kMoeStride;
 #pragma unroll
-        for (int i = 0; i < 2; ++i) *reinterpret_cast<uint4*>(&Bs[(tid >> 2) + 32 * i][ac]) = b_reg[i];
-        __syncthreads();
-        if (k0 + MK < K) fetch(k0 + MK, a_reg, b_reg);
-#pragma unroll
-        for (int kk = 0; kk < MK / 16; ++kk) {
-            uint32_t a[2][4], b[2][2];
-            const int c = kk * 16 + (lane & 3) * 2;
+        for (int ks = 0; ks < MK / 16; ++ks) {
+            uint32_t b[4];
+            qi_attn::ldmatrix_x4(bs + (warp * 16 + (lane & 7) + (lane >> 4) * 8) * kMoeStride + ((ks * 2 + ((lane >> 3) & 1)) << 4), b[0], b[1], b[2], b[3]);
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
-                const int r = i * 16 + (lane >> 2);
-                a[i][0] = *reinterpret_cast<const uint32_t*>(&As[r][c]);
-                a[i][1] = *reinterpret_cast<const uint32_t*>(&As[r + 8][c]);
-                a[i][2] = *reinterpret_cast<const uint32_t*>(&As[r][c + 8]);
-                a[i][3] = *reinterpret_cast<const uint32_t*>(&As[r + 8][c + 8]);
+                if (i < m_tiles) {
+                    uint32_t a[4];
+                    qi_attn::ldmatrix_x4(as + (i * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kMoeStride + ((ks * 2 + (lane >> 4)) << 4), a[0], a[1], a[2], a[3]);
+                    qi_attn::mma_bf16(acc[i][0], a, b[0], b[1]);
+                    qi_attn::mma_bf16(acc[i][1], a, b[2], b[3]);
+                }
             }
-#pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                const int nn = warp * 16 + j * 8 + (lane >> 2);
-                b[j][0] = *reinterpret_cast<const uint32_t*>(&Bs[nn][c]);
-                b[j][1] = *reinterpret_cast<const uint32_t*>(&Bs[nn][c + 8]);
-            }
-#pragma unroll
-            for (int i = 0; i < 2; ++i)
-#pragma unroll
-                for (int j = 0; j < 2; ++j) mma_bf16_16816(acc[i][j], a[i][0], a[i][1], a[i][2], a[i][3], b[j][0], b[j][1]);
         }
     }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
 #pragma unroll
     for (int i = 0; i < 2; ++i)
 #pragma unroll
@@ -306,9 +303,9 @@ moe_gemm_mma_kernel(const qi::bf16* __restrict__ x, const qi::bf16* __restrict__
                 const int m = i * 16 + (lane >> 2) + 8 * half;
                 if (m >= rows) continue;
                 if (epilogue) {      // n is even: this thread's two columns are a (gate, up) pair
-                    const float w = pair_scale ? pair_scale[order[row0 + m]] : 1.f;
+                    const float s = pair_scale ? pair_scale[order[row0 + m]] : 1.f;
                     if (n + 1 < N)
-                        y[(size_t)(row0 + m) * ldy + (n >> 1)] = __float2bfloat16_rn(scaled_silu_mul(acc[i][j][2 * half], acc[i][j][2 * half + 1], w));
+                        y[(size_t)(row0 + m) * ldy + (n >> 1)] = __float2bfloat16_rn(scaled_silu_mul(acc[i][j][2 * half], acc[i][j][2 * half + 1], s));
                     continue;
                 }
                 qi::bf16* dst = y + (size_t)(row0 + m) * ldy + n;
@@ -505,8 +502,15 @@ extern "C" int qi_moe_gemm(const void* x, int x_dtype, const void* w, int w_dtyp
     QI_REQUIRE(ldx >= K && ldy >= (epilogue ? N / 2 : N), "moe_gemm: a leading dimension is smaller than its row");
     QI_REQUIRE(max_tiles <= 65535, "moe_gemm: %d row tiles are too many for one launch", max_tiles);
     if (max_tiles == 0) return 0;
-    if (x_dtype == qi::kBF16 && w_dtype == qi::kBF16 && y_dtype == qi::kBF16 && K % 8 == 0 && ldx % 8 == 0) {
-        qi::launch(moe_gemm_mma_kernel, dim3((N + MN - 1) / MN, max_tiles), dim3(128), 0, stream, (const qi::bf16*)x,
+    if (x_dtype == qi::kBF16 && w_dtype == qi::kBF16 && y_dtype == qi::kBF16 && K % 8 == 0 && ldx % 8 == 0 &&
+        (((uintptr_t)x | (uintptr_t)w) & 15) == 0) {
+        static bool configured = false;
+        if (!configured) {
+            if (cudaFuncSetAttribute(moe_gemm_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kMoeSmem) != cudaSuccess)
+                return qi::fail("moe_gemm: %d bytes of shared memory were refused", kMoeSmem);
+            configured = true;
+        }
+        qi::launch(moe_gemm_mma_kernel, dim3((N + MN - 1) / MN, max_tiles), dim3(128), kMoeSmem, stream, (const qi::bf16*)x,
                    (const qi::bf16*)w, (qi::bf16*)y, tiles, order, top, gather, N, K, ldx, ldy, n_src, n_rows, E, epilogue,
                    pair_scale);
         return qi::check_launch("moe_gemm_mma");
